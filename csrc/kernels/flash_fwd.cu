@@ -36,6 +36,7 @@ struct FlashFwdParams {
   // point at peer memory) are visited in one pass; queries and keys carry global positions (contiguous split, or
   // zigzag: rank r holds sequence chunks r and 2W-1-r of 2W).  cp_world == 1 is plain attention.
   int cp_world, cp_rank, zigzag;
+  int window;   // causal only: a query sees its own position and the window - 1 before it; 0 = no limit
 };
 
 constexpr int kFaMaxRanks = 8;
@@ -152,6 +153,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         if (p.causal) {
           const int vis = q_last < kbase ? 0 : (q_last - kbase) / kFaBlockKV + 1;
           nb = nb < vis ? nb : vis;
+        }
+        if (p.window > 0 && p.cp_world == 1) {
+          // blocks that end before the first query's window are skipped
+          const int first = max(0, q_base - p.window + 1) / kFaBlockKV;
+          kv0 += first * kFaBlockKV;
+          kbase += first * kFaBlockKV;
+          nb -= first;
         }
         if (nb > 0) {
           segs[ns] = KvSeg{nb, o, kv0, kbase};
@@ -313,6 +321,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const uint32_t lane_base = uint32_t(quarter * 32) << 16;
     const uint32_t o_mine = tmem_base + lane_base + Cfg::kColO + grp * D;
     float m_used = 0.f, l = 0.f;
+    bool seen = false;   // this row has met a visible key (with a window, whole blocks may lie before it)
     bool ok = true;
     const bool tr = p.trace != nullptr && blockIdx.z == 0 && h == 0 && b == 0 && warp == 2 && lane == 0;
     long long tc[6] = {0, 0, 0, 0, 0, 0};
@@ -332,6 +341,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       // last visible column of this 128-key block for this row: causal position and end of the rank's keys
       int limit = p.Tk - 1 - kv0b;
       if (p.causal) limit = min(limit, q_base + row - kbase);
+      const int lower = p.window > 0 ? q_base + row - kbase - p.window + 1 : 0;   // first visible column
       const uint32_t s_mine = tmem_base + lane_base + Cfg::kColS + sb * 128;
       // pass 1: row maximum (the scores are read from tensor memory twice, 64 columns at a time, instead of
       // holding all 128 in registers)
@@ -342,7 +352,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         tmem_ld_32x32(s_mine + hh * 64, r[0]);
         tmem_ld_32x32(s_mine + hh * 64 + 32, r[1]);
         tmem_ld_wait();
-        if (limit >= hh * 64 + 63) {
+        if (limit >= hh * 64 + 63 && lower <= hh * 64) {
 #pragma unroll
           for (int c = 0; c < 2; ++c)
 #pragma unroll
@@ -352,14 +362,17 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           for (int c = 0; c < 2; ++c)
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              if (hh * 64 + c * 32 + i <= limit) mx = fmaxf(mx, __uint_as_float(r[c][i]));
+              if (hh * 64 + c * 32 + i <= limit && hh * 64 + c * 32 + i >= lower) mx = fmaxf(mx, __uint_as_float(r[c][i]));
         }
       }
       if (tr) { const long long c1 = clock64(); tc[1] += c1 - c0; c0 = c1; }   // pass 1 (row maximum)
       const float m_blk = mx * p.scale_log2;
-      if (j == grp) {
+      if (!seen) {
+        // nothing accumulated for this row yet (its P entries were zero): take the block's maximum as it is
         m_used = (m_blk == -INFINITY) ? 0.f : m_blk;
-      } else {
+        seen = m_blk != -INFINITY;
+      }
+      if (j != grp) {
         const float m_new = fmaxf(m_used, m_blk);
         const bool need = (m_new - m_used > 8.f);
         if (__any_sync(0xffffffffu, need)) {
@@ -396,13 +409,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         tmem_ld_32x32(s_mine + hh * 64, r[0]);
         tmem_ld_32x32(s_mine + hh * 64 + 32, r[1]);
         tmem_ld_wait();
-        const bool full_vis = (limit >= hh * 64 + 63);
+        const bool full_vis = (limit >= hh * 64 + 63 && lower <= hh * 64);
 #pragma unroll
         for (int c = 0; c < 2; ++c)
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             float pv = ex2_approx_f(fmaf(__uint_as_float(r[c][i]), p.scale_log2, -m_used));
-            if (!full_vis && hh * 64 + c * 32 + i > limit) pv = 0.f;
+            if (!full_vis && (hh * 64 + c * 32 + i > limit || hh * 64 + c * 32 + i < lower)) pv = 0.f;
             sum += pv;
             r[c][i] = __float_as_uint(pv);
           }
@@ -453,11 +466,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     }
     if (ok) {
       float m_all = m_used, a_mine = 1.f, a_other = 0.f;
-      if (mine_used && other_used) {
+      if (mine_used && other_used && l > 0.f && l_o > 0.f) {
         m_all = fmaxf(m_used, m_o);
         a_mine = ex2_approx_f(m_used - m_all);
         a_other = ex2_approx_f(m_o - m_all);
-      } else if (!mine_used && other_used) {
+      } else if (other_used && !(mine_used && l > 0.f)) {     // only the other group met a visible key of this row
         m_all = m_o; a_mine = 0.f; a_other = 1.f;
       }
       const float l_all = (mine_used ? l * a_mine : 0.f) + (other_used ? l_o * a_other : 0.f);
@@ -530,7 +543,8 @@ static int launch_flash_fwd(const CUtensorMap& tq, const KvMaps& maps, const Fla
 static int flash_fwd_common(const void* q, const void* const* k_ptrs, const void* const* v_ptrs, void* o, float* lse, int B,
                             int Tq, int Tk, int Hq, int Hkv, int D, long long sq_b, long long sq_t, long long sk_b,
                             long long sk_t, long long sv_b, long long sv_t, long long so_b, long long so_t, float scale,
-                            int causal, int cp_world, int cp_rank, int zigzag, void* stream) {
+                            int causal, int cp_world, int cp_rank, int zigzag, int window, void* stream) {
+  if (window < 0 || (window > 0 && (!causal || cp_world != 1))) return -int(kStatusBadArgument);
   if ((D != 64 && D != 128) || Hq % Hkv != 0 || cp_world < 1 || cp_world > kFaMaxRanks) return -int(kStatusBadArgument);
   if (cp_world > 1 && zigzag && ((Tq / 2) % kFaBlockQ != 0 || (Tk / 2) % kFaBlockKV != 0)) return -int(kStatusBadArgument);
   if (cp_world > 1 && !zigzag && (Tq % kFaBlockQ != 0 || Tk % kFaBlockKV != 0)) return -int(kStatusBadArgument);
@@ -556,6 +570,7 @@ static int flash_fwd_common(const void* q, const void* const* k_ptrs, const void
   p.scale_log2 = scale * 1.4426950408889634f;
   p.causal = causal;
   p.cp_world = cp_world; p.cp_rank = cp_rank; p.zigzag = zigzag;
+  p.window = window;
   p.status = device_status_word();
   p.trace = g_fwd_trace;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -578,7 +593,18 @@ int lt_flash_fwd(const void* q, const void* k, const void* v, void* o, float* ls
   const void* ks[1] = {k};
   const void* vs[1] = {v};
   return lt::flash_fwd_common(q, ks, vs, o, lse, B, Tq, Tk, Hq, Hkv, D, sq_b, sq_t, sk_b, sk_t, sv_b, sv_t, so_b, so_t, scale,
-                              causal, 1, 0, 0, stream);
+                              causal, 1, 0, 0, 0, stream);
+}
+
+// Causal attention in which query i sees key j only when 0 <= i - j < window (positions counted as in lt_flash_fwd, the
+// last query on the last key): key blocks outside every row's window are never loaded.
+int lt_flash_fwd_window(const void* q, const void* k, const void* v, void* o, float* lse, int B, int Tq, int Tk, int Hq, int Hkv,
+                        int D, long long sq_b, long long sq_t, long long sk_b, long long sk_t, long long sv_b, long long sv_t,
+                        long long so_b, long long so_t, float scale, int window, void* stream) {
+  const void* ks[1] = {k};
+  const void* vs[1] = {v};
+  return lt::flash_fwd_common(q, ks, vs, o, lse, B, Tq, Tk, Hq, Hkv, D, sq_b, sq_t, sk_b, sk_t, sv_b, sv_t, so_b, so_t, scale,
+                              1, 1, 0, 0, window, stream);
 }
 
 // Context-parallel forward: k_ptrs[r] / v_ptrs[r] are rank r's KV shards [B, Tk, Hkv, D] (peer-mapped pointers, all with
@@ -589,7 +615,7 @@ int lt_flash_fwd_cp(const void* q, const void* const* k_ptrs, const void* const*
                     long long sv_b, long long sv_t, long long so_b, long long so_t, float scale, int causal, int cp_world,
                     int cp_rank, int zigzag, void* stream) {
   return lt::flash_fwd_common(q, k_ptrs, v_ptrs, o, lse, B, Tq, Tk, Hq, Hkv, D, sq_b, sq_t, sk_b, sk_t, sv_b, sv_t, so_b, so_t,
-                              scale, causal, cp_world, cp_rank, zigzag, stream);
+                              scale, causal, cp_world, cp_rank, zigzag, 0, stream);
 }
 
 }  // extern "C"

@@ -166,6 +166,32 @@ int lt_gemm_e4m3(const void* A, const void* B, void* C, int M, int N, int K, lon
                      a_scale, b_scale);
 }
 
+// C[M, blocks * nb] (fp32) = A[M, blocks * K] @ blockdiag(B_0 .. )^T with B [blocks, nb, K]: columns z * nb .. of C are the
+// product of columns z * K .. of A with block z.  bf16 operands, K a multiple of 8, nb a multiple of 128.
+int lt_gemm_block_diag(const void* A, const void* B, float* C, int M, int blocks, int nb, int K, long long lda, long long ldc,
+                       void* stream) {
+  using namespace lt;
+  if (M <= 0 || blocks <= 0) return 0;
+  if ((K & 7) || nb % 128 != 0 || (lda & 7) || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15))
+    return -int(kStatusBadArgument);
+  const int block_n = nb % 256 == 0 ? 256 : 128;
+  GemmParams p{};
+  p.M = M; p.N = blocks * nb; p.K = K;
+  p.C = C; p.ldc = ldc; p.out_fp32 = 1; p.alpha = 1.f;
+  p.status = device_status_word();
+  p.diag_n = nb;
+  fill_tiles(p, block_n);
+  CUtensorMap tmA, tmB;
+  int r = encode_tmap_2d(&tmA, A, 2, uint64_t(blocks) * K, (uint64_t)M, (uint64_t)lda * 2, kBlockK, kBlockM, 1);
+  if (r) return 1000 + r;
+  r = encode_tmap_2d(&tmB, B, 2, (uint64_t)K, uint64_t(blocks) * nb, (uint64_t)K * 2, kBlockK, block_n, 1);
+  if (r) return 2000 + r;
+  int grid = sm_count();
+  if (grid > p.num_tiles) grid = p.num_tiles;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return block_n == 256 ? launch_gemm<256, 0, 0>(tmA, tmB, p, grid, st) : launch_gemm<128, 0, 0>(tmA, tmB, p, grid, st);
+}
+
 static int gemm_launch(int kind, const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
                        long long ldc, int a_major, int b_major, int out_fp32, const void* bias, const void* residual,
                        long long ldr, int act, int accumulate, float alpha, int block_n, int max_ctas, void* stream,

@@ -78,6 +78,9 @@ struct GemmParams {
   // times b_scale[c] (fp32, nullptr: 1).
   const float* a_scale;
   const float* b_scale;
+  // Block-diagonal B (one-CTA kernel, both operands K-major): columns come in groups of diag_n, and group z multiplies the K
+  // columns of A that start at z * K.  A's tensor map spans all groups; a K tile that runs past K meets zeros of B.  0: off.
+  int diag_n;
 };
 
 struct WorkItem {
@@ -361,7 +364,8 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensor
           const uint32_t a_dst = smem_base + stage * Cfg::kStageBytes;
           const uint32_t b_dst = a_dst + Cfg::kABytes;
           if (A_MAJOR == 0) {
-            tma_load_2d(a_dst, tmA, fb, kb * kBlockK, m_blk * kBlockM);
+            const int a_off = p.diag_n > 0 ? (n_blk * BLOCK_N / p.diag_n) * p.K : 0;
+            tma_load_2d(a_dst, tmA, fb, a_off + kb * kBlockK, m_blk * kBlockM);
           } else {
 #pragma unroll
             for (int i = 0; i < kBlockM / 64; ++i)

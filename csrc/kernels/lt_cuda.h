@@ -47,6 +47,9 @@ int lt_flash_fwd_cp(const void* q, const void* const* k_ptrs, const void* const*
                     int Tq, int Tk, int Hq, int Hkv, int D, long long sq_b, long long sq_t, long long sk_b,
                     long long sk_t, long long sv_b, long long sv_t, long long so_b, long long so_t, float scale,
                     int causal, int cp_world, int cp_rank, int zigzag, void* stream);
+int lt_flash_fwd_window(const void* q, const void* k, const void* v, void* o, float* lse, int B, int Tq, int Tk, int Hq,
+                        int Hkv, int D, long long sq_b, long long sq_t, long long sk_b, long long sk_t, long long sv_b,
+                        long long sv_t, long long so_b, long long so_t, float scale, int window, void* stream);
 
 // ---- fsdp_fused.cu: ZeRO-3 fused paths: all-gather -> GEMM, reduce-scatter -> AdamW, shard gathers, flag barrier between ranks
 int lt_ag_gemm_bf16(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
@@ -96,6 +99,8 @@ int lt_gemm_typed(int kind, const void* A, const void* B, void* C, int M, int N,
 int lt_gemm_e4m3(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
                  long long ldc, int out_fp32, const float* a_scale, const float* b_scale, const void* bias,
                  const void* residual, long long ldr, int act, float alpha, void* stream);
+int lt_gemm_block_diag(const void* A, const void* B, float* C, int M, int blocks, int nb, int K, long long lda,
+                       long long ldc, void* stream);
 
 // ---- gemv.cu: GEMV for 1-8 rows
 int lt_gemv_bf16(const void* x, long long ldx, const void* w, long long ldw, void* y, long long ldy,
@@ -166,11 +171,61 @@ int lt_norm_bwd_noalloc(int layer_norm, const void* dy, const void* x, const voi
                         const float* rstd, const void* dres, void* dx, void* dw, void* db, int grads_fp32,
                         int accumulate, int M, int D, void* stream);
 
+// ---- hyper_norm.cu: residual streams mixed by hyper-connections, with the RMS norm of the next sublayer
+int lt_hyper_norm(int fp32, void* x, const int* tokens, const void* embed, const void* y1, long long ldy1, const float* n1,
+                  const void* y2, long long ldy2, const float* n2, const float* mix, const float* out, const float* in,
+                  const float* norm, float eps, void* h, long long ldh, const int* rows, int n_rows, int width, int streams,
+                  int write_x, void* stream);
+
+// ---- gemm_simt.cu: CUDA-core GEMM (true fp32, odd shapes, batches) and narrow projections with fp32 results
+int lt_gemm_simt(int in_fp32, int out_fp32, const void* A, const void* B, void* C, int M, int N, int K, long long lda,
+                 long long ldb, long long ldc, int batch, long long sa, long long sb, long long sc, float alpha, void* stream);
+int lt_rows_dot(int fp32, const void* x, long long ldx, const void* w, float* y, int R, int J, int K, void* stream);
+
+// ---- window_attn.cu: projection norm + rotary embedding + cache write, window gather, CUDA-core attention, head gates
+int lt_qkv_rope(int fp32, const void* proj, long long ld, int n, int q_off, int k_off, int v_off, int H, int G, int D, int E,
+                int DP, int EP, const float* q_norm, const float* k_norm, float eps, const int* positions, const int* slots,
+                const double* freq, int rot_dims, float gain, void* q_out, void* k_cache, void* v_cache, int block_size,
+                void* k_lin, void* v_lin, void* stream);
+int lt_kv_gather(const void* k_cache, const void* v_cache, void* k_lin, void* v_lin, const int* table, int pos0, int n, int G,
+                 int k_bytes, int v_bytes, int block_size, void* stream);
+int lt_window_attn(int fp32, const void* q, const void* k_cache, const void* v_cache, const int* tables, long long table_stride,
+                   const int* positions, void* o, const void* gate, long long ldg, int N, int H, int G, int D, int E, int DP,
+                   int EP, int block_size, int window, float scale, void* stream);
+int lt_head_gate(int fp32, const void* o, const void* gate, long long ldg, void* out, long long rows, int H, int E, int EP,
+                 void* stream);
+
+// ---- rglru.cu: causal convolution and gated linear recurrence, prompt scan and decode step
+int lt_conv_causal(int fp32, const void* x, long long ldx, const float* xb, const float* w, const float* b, const float* ring,
+                   void* u, int N, int C, int taps, int start, void* stream);
+int lt_rglru_scan(int fp32, const void* u, const float* gates, const float* rb, const float* ib, const float* sp, const void* y,
+                  long long ldy, const float* yb, const void* x, long long ldx, const float* xb, float* state, float* ring,
+                  void* out, int N, int C, int bw, int taps, int start, void* stream);
+int lt_rglru_step(int fp32, const void* x, long long ldx, const float* xb, const float* conv_w, const float* conv_b,
+                  const void* gates, const float* rb, const float* ib, const float* sp, const void* y, long long ldy,
+                  const float* yb, float* state, float* ring, const int* slots, const int* positions, void* out, int S, int C,
+                  int bw, int taps, void* stream);
+
+// ---- mlstm.cu: matrix memory with exponential gates, chunked prompt kernels and decode step
+int lt_mlstm_prefill(const void* q, const void* k, const void* v, long long ld, const float* logits, const float* ib,
+                     const float* fb, float cap, float qscale, const float* norm, float eps, const void* gate, long long ldg,
+                     float* S, float* n, float* m, float* a, float* f, float* cmax, float* m_start, float* U, float* nU, float* o,
+                     void* out, int N, int H, int D, int E, int start, void* stream);
+int lt_mlstm_step(int fp32, const void* q, const void* k, const void* v, long long ld, const float* logits, const float* ib,
+                  const float* fb, float cap, float qscale, float* S, float* n, float* m, const int* slots, const int* positions,
+                  float* o, int rows, int H, int D, int E, int seq_len, int slot, int start, void* stream);
+int lt_head_norm_gate(int fp32, const float* o, const float* w, const void* gate, long long ldg, void* out, long long rows, int H,
+                      int E, float eps, void* stream);
+
 // ---- paged_decode.cu: decode attention over a block-paged KV cache, cache append
 int lt_paged_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                     const int* context_lens, float* part, void* o, int S, int Hq, int Hkv, int D, int block_size,
                     int max_blocks, int num_blocks, int splits, float scale, int kv_fp8, float k_scale, float v_scale,
                     void* stream);
+int lt_paged_decode_window(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
+                           const int* context_lens, float* part, void* o, int S, int Hq, int Hkv, int D, int block_size,
+                           int max_blocks, int num_blocks, int splits, float scale, int kv_fp8, float k_scale,
+                           float v_scale, int window, const void* gate, long long ldg, int vdim, void* stream);
 int lt_kv_append(const void* k_new, const void* v_new, void* k_cache, void* v_cache, const int* slots, long long n_tok,
                  int Hkv, int D, int block_size, int kv_fp8, float k_scale, float v_scale, void* stream);
 
@@ -178,6 +233,7 @@ int lt_kv_append(const void* k_new, const void* v_new, void* k_cache, void* v_ca
 int lt_rope(void* x, const float* cos_t, const float* sin_t, const int* pos, long long rows, int T, int heads, int hd,
             long long row_stride, int backward, void* stream);
 int lt_swiglu_fwd(const void* gu, void* h, long long M, int F, void* stream);
+int lt_clamped_glu(int fp32, const void* gu, void* h, long long M, int F, float limit, float slope, void* stream);
 int lt_swiglu_bwd(const void* gu, const void* dh, void* dgu, long long M, int F, void* stream);
 int lt_gelu_fwd(const void* x, void* y, long long n, void* stream);
 int lt_gelu_bwd(const void* x, const void* dy, void* dx, long long n, void* stream);

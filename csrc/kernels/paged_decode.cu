@@ -46,7 +46,7 @@ template <int D, bool FP8>
 __global__ void paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict__ k_cache,
                                     const void* __restrict__ v_cache, const int* __restrict__ block_tables,
                                     const int* __restrict__ context_lens, float* __restrict__ part, int S, int Hq, int Hkv,
-                                    int block_size, int max_blocks, int splits, float scale, float k_scale, float v_scale) {
+                                    int block_size, int max_blocks, int splits, float scale, float k_scale, float v_scale, int window) {
   constexpr int E = D / 32;
   const int warp_global = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
@@ -57,8 +57,9 @@ __global__ void paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const v
   const int s = warp_global / (splits * Hq);
   const int hkv = h / (Hq / Hkv);
   const int ctx = context_lens[s];
-  const int per = (ctx + splits - 1) / splits;
-  const int t0 = sp * per, t1 = min(ctx, t0 + per);
+  const int lo = window > 0 ? max(0, ctx - window) : 0;              // first visible key
+  const int per = (ctx - lo + splits - 1) / splits;
+  const int t0 = lo + sp * per, t1 = min(ctx, t0 + per);
   float qv[E];
   {
     const __nv_bfloat16* qp = q + ((long long)s * Hq + h) * D + lane * E;
@@ -354,7 +355,7 @@ __global__ void __launch_bounds__(kPdWarps * 32)
 paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                         const __nv_bfloat16* __restrict__ q, const int* __restrict__ block_tables,
                         const int* __restrict__ context_lens, float* __restrict__ part, int S, int Hq, int Hkv, int block_size,
-                        int max_blocks, int splits, float scale, int* status) {
+                        int max_blocks, int splits, float scale, int window, int* status) {
   using Cfg = PdMmaCfg<D>;
   constexpr int ST = Cfg::kStages;
   constexpr int KS = D / 16;     // k-steps of the score product
@@ -393,8 +394,10 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
   __syncthreads();
   volatile int* abort_flag = &abort_s;
   const int ctx = context_lens[s];
-  const int per = ((ctx + splits - 1) / splits + 31) / 32 * 32;      // whole 32-key chunks per split
-  const int t0 = sp * per, t1 = min(ctx, t0 + per);
+  const int lo = window > 0 ? max(0, ctx - window) : 0;              // first visible key
+  const int base = lo & ~31;                                         // chunks start on multiples of 32 keys
+  const int per = ((ctx - base + splits - 1) / splits + 31) / 32 * 32;      // whole 32-key chunks per split
+  const int t0 = base + sp * per, t1 = min(ctx, t0 + per);
   const int* bt = block_tables + (long long)s * max_blocks;
   const int n_chunks = t1 > t0 ? (t1 - t0 + 31) / 32 : 0;
   const int my_n = n_chunks > warp ? (n_chunks - warp + kPdWarps - 1) / kPdWarps : 0;   // chunks warp, warp + 4, ...
@@ -480,7 +483,8 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
     for (int t = 0; t < 4; ++t) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const bool live = t * 8 + qd * 2 + e < nk;
+        const int col = t * 8 + qd * 2 + e;
+        const bool live = col < nk && c0 + col >= lo;
         sacc[t][e] = live ? sacc[t][e] * scale : -INFINITY;
         sacc[t][2 + e] = live ? sacc[t][2 + e] * scale : -INFINITY;
         mx_lo = fmaxf(mx_lo, sacc[t][e]);
@@ -491,7 +495,7 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
     mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
     mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
     mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
-    const float nm_lo = fmaxf(m_lo, mx_lo), nm_hi = fmaxf(m_hi, mx_hi);   // finite: every chunk has a live key
+    const float nm_lo = fmaxf(m_lo, mx_lo), nm_hi = fmaxf(m_hi, mx_hi);   // finite: every chunk has a live key (the first one ends after `lo`)
     const float a_lo = (m_lo == -INFINITY) ? 0.f : __expf(m_lo - nm_lo);
     const float a_hi = (m_hi == -INFINITY) ? 0.f : __expf(m_hi - nm_hi);
     m_lo = nm_lo; m_hi = nm_hi;
@@ -572,7 +576,8 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
 }
 
 template <int D>
-__global__ void paged_decode_merge_kernel(const float* __restrict__ part, __nv_bfloat16* __restrict__ o, int rows, int splits) {
+__global__ void paged_decode_merge_kernel(const float* __restrict__ part, __nv_bfloat16* __restrict__ o, int rows, int splits,
+                                          const __nv_bfloat16* __restrict__ gate, long long ldg, int Hq, int vdim) {
   const int row = blockIdx.x * (blockDim.x / 32) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (row >= rows) return;
@@ -591,9 +596,11 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part, __nv_b
 #pragma unroll
     for (int i = 0; i < E; ++i) acc[i] += w * p[lane * E + i];
   }
-  const float inv = wsum > 0.f ? 1.f / wsum : 0.f;
+  float inv = wsum > 0.f ? 1.f / wsum : 0.f;
+  if (gate) inv /= 1.f + expf(-__bfloat162float(gate[(row / Hq) * ldg + row % Hq]));     // times sigmoid(gate) of this head
 #pragma unroll
-  for (int i = 0; i < E; ++i) o[(long long)row * D + lane * E + i] = __float2bfloat16(acc[i] * inv);
+  for (int i = 0; i < E; ++i)
+    if (lane * E + i < vdim) o[(long long)row * vdim + lane * E + i] = __float2bfloat16(acc[i] * inv);
 }
 
 // slot = block * block_size + offset for each new token.
@@ -630,8 +637,19 @@ extern "C" {
 int lt_paged_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_tables, const int* context_lens,
                     float* part, void* o, int S, int Hq, int Hkv, int D, int block_size, int max_blocks, int num_blocks,
                     int splits, float scale, int kv_fp8, float k_scale, float v_scale, void* stream) {
+  return lt_paged_decode_window(q, k_cache, v_cache, block_tables, context_lens, part, o, S, Hq, Hkv, D, block_size, max_blocks,
+                                num_blocks, splits, scale, kv_fp8, k_scale, v_scale, 0, nullptr, 0, D, stream);
+}
+
+// The same over the newest `window` keys of every sequence (0: all of them), with an optional gate per head (logits
+// gate[s * ldg + h]; the head's output is multiplied by its sigmoid) and only the first vdim of the D value columns
+// written: o is [S, Hq, vdim].
+int lt_paged_decode_window(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
+                           const int* context_lens, float* part, void* o, int S, int Hq, int Hkv, int D, int block_size,
+                           int max_blocks, int num_blocks, int splits, float scale, int kv_fp8, float k_scale, float v_scale,
+                           int window, const void* gate, long long ldg, int vdim, void* stream) {
   using namespace lt;
-  if ((D != 64 && D != 128) || Hq % Hkv != 0 || splits < 1) return -int(kStatusBadArgument);
+  if ((D != 64 && D != 128) || Hq % Hkv != 0 || splits < 1 || window < 0 || vdim < 1 || vdim > D) return -int(kStatusBadArgument);
   if (S == 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int warps = S * Hq * splits;
@@ -640,7 +658,7 @@ int lt_paged_decode(const void* q, const void* k_cache, const void* v_cache, con
   auto Q = static_cast<const __nv_bfloat16*>(q);
 #define LT_PD(DD, F8) \
   paged_decode_kernel<DD, F8><<<blocks, threads, 0, st>>>(Q, k_cache, v_cache, block_tables, context_lens, part, S, Hq, Hkv, \
-                                                          block_size, max_blocks, splits, scale, k_scale, v_scale)
+                                                          block_size, max_blocks, splits, scale, k_scale, v_scale, window)
   const int G = Hq / Hkv;
   const bool bs_ok = block_size > 0 && (32 % block_size == 0 || block_size % 32 == 0);
   const bool aligned = (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0 && (reinterpret_cast<uintptr_t>(v_cache) & 15) == 0;
@@ -661,9 +679,9 @@ int lt_paged_decode(const void* q, const void* k_cache, const void* v_cache, con
     if (r == 0) r = encode_tmap_2d(&tmV, v_cache, 2, D, rows, uint64_t(D) * 2, 64, run, 1);
     if (r) return r > 0 ? 1000 + r : r;
     int* status = device_status_word();
-    if (D == 64) paged_decode_mma_kernel<64><<<ctas, kPdWarps * 32, PdMmaCfg<64>::kSmemBytes, st>>>(tmK, tmV, Q, block_tables, context_lens, part, S, Hq, Hkv, block_size, max_blocks, splits, scale, status);
-    else paged_decode_mma_kernel<128><<<ctas, kPdWarps * 32, PdMmaCfg<128>::kSmemBytes, st>>>(tmK, tmV, Q, block_tables, context_lens, part, S, Hq, Hkv, block_size, max_blocks, splits, scale, status);
-  } else if (!kv_fp8 && G <= kPdMaxG && bs_ok && (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0 && (reinterpret_cast<uintptr_t>(v_cache) & 15) == 0) {
+    if (D == 64) paged_decode_mma_kernel<64><<<ctas, kPdWarps * 32, PdMmaCfg<64>::kSmemBytes, st>>>(tmK, tmV, Q, block_tables, context_lens, part, S, Hq, Hkv, block_size, max_blocks, splits, scale, window, status);
+    else paged_decode_mma_kernel<128><<<ctas, kPdWarps * 32, PdMmaCfg<128>::kSmemBytes, st>>>(tmK, tmV, Q, block_tables, context_lens, part, S, Hq, Hkv, block_size, max_blocks, splits, scale, window, status);
+  } else if (!kv_fp8 && window == 0 && G <= kPdMaxG && bs_ok && (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0 && (reinterpret_cast<uintptr_t>(v_cache) & 15) == 0) {
     // bf16 caches: every K / V byte is read once for the whole group of query heads, through a shared-memory pipeline
     const int ctas = S * Hkv * splits;
     auto KC = static_cast<const __nv_bfloat16*>(k_cache);
@@ -683,8 +701,10 @@ int lt_paged_decode(const void* q, const void* k_cache, const void* v_cache, con
   LT_LAUNCH_CHECK();
   const int rows = S * Hq;
   const int mb = (rows + 3) / 4;
-  if (D == 64) paged_decode_merge_kernel<64><<<mb, 128, 0, st>>>(part, static_cast<__nv_bfloat16*>(o), rows, splits);
-  else paged_decode_merge_kernel<128><<<mb, 128, 0, st>>>(part, static_cast<__nv_bfloat16*>(o), rows, splits);
+  auto O = static_cast<__nv_bfloat16*>(o);
+  auto GT = static_cast<const __nv_bfloat16*>(gate);
+  if (D == 64) paged_decode_merge_kernel<64><<<mb, 128, 0, st>>>(part, O, rows, splits, GT, ldg, Hq, vdim);
+  else paged_decode_merge_kernel<128><<<mb, 128, 0, st>>>(part, O, rows, splits, GT, ldg, Hq, vdim);
   LT_LAUNCH_CHECK();
   return 0;
 }

@@ -9,6 +9,7 @@
 #include "lt_cuda.h"
 #include "common/host.h"
 #include "common/ptx.cuh"
+#include "common/scalar.cuh"
 
 namespace lt {
 
@@ -73,6 +74,39 @@ __global__ void swiglu_fwd_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfl
   }
 }
 // dgu may alias gu (written in place).
+// h = g sigmoid(slope g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); gu rows are [gate | up].
+template <typename T>
+__global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ h, long long M, int F, float limit, float slope) {
+  const long long total = M * F;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / F, c = i % F;
+    const float g = fminf(ldf(gu + r * 2 * F + c), limit);
+    const float u = fminf(fmaxf(ldf(gu + r * 2 * F + F + c), -limit), limit);
+    stf(h + i, g * sigmoid_f(slope * g) * (u + 1.f));
+  }
+}
+
+// The same for bf16, eight columns per thread.
+__global__ void clamped_glu8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ h, long long M, int F,
+                                    float limit, float slope) {
+  const int fu = F / 8;
+  const long long total = M * fu;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / fu, c = (i % fu) * 8;
+    const uint4 gv = *reinterpret_cast<const uint4*>(gu + r * 2 * F + c), uv = *reinterpret_cast<const uint4*>(gu + r * 2 * F + F + c);
+    const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w}, uw[4] = {uv.x, uv.y, uv.z, uv.w};
+    uint32_t o[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 g2 = unpack_bf16x2(gw[k]), u2 = unpack_bf16x2(uw[k]);
+      const float g0 = fminf(g2.x, limit), g1 = fminf(g2.y, limit);
+      const float u0 = fminf(fmaxf(u2.x, -limit), limit), u1 = fminf(fmaxf(u2.y, -limit), limit);
+      o[k] = pack_bf16x2(g0 * sigmoid_f(slope * g0) * (u0 + 1.f), g1 * sigmoid_f(slope * g1) * (u1 + 1.f));
+    }
+    *reinterpret_cast<uint4*>(h + r * F + c) = make_uint4(o[0], o[1], o[2], o[3]);
+  }
+}
+
 __global__ void swiglu_bwd_kernel(const __nv_bfloat16* gu, const __nv_bfloat16* __restrict__ dh, __nv_bfloat16* dgu,
                                   long long M, int F) {
   const int vpr = F / 8;
@@ -225,6 +259,16 @@ int lt_swiglu_fwd(const void* gu, void* h, long long M, int F, void* stream) {
   if (M == 0) return 0;
   swiglu_fwd_kernel<<<grid_for(M * (F / 8), 256), 256, 0, static_cast<cudaStream_t>(stream)>>>(
       static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(h), M, F);
+  LT_LAUNCH_CHECK();
+  return 0;
+}
+int lt_clamped_glu(int fp32, const void* gu, void* h, long long M, int F, float limit, float slope, void* stream) {
+  using namespace lt;
+  if (M == 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (fp32) clamped_glu_kernel<float><<<grid_for(M * F, 256), 256, 0, st>>>(static_cast<const float*>(gu), static_cast<float*>(h), M, F, limit, slope);
+  else if (F % 8 == 0) clamped_glu8_kernel<<<grid_for(M * (F / 8), 256), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(h), M, F, limit, slope);
+  else clamped_glu_kernel<__nv_bfloat16><<<grid_for(M * F, 256), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(h), M, F, limit, slope);
   LT_LAUNCH_CHECK();
   return 0;
 }

@@ -96,6 +96,10 @@ int lt_sched_plan(void* h, int64_t* req_ids, int32_t* chunk_start, int32_t* chun
 int lt_sched_commit(void* h, int64_t id, int32_t token);
 int lt_sched_tokens(void* h, int64_t id, int32_t* out, int cap, int* prompt_len);
 int lt_sched_block_table(void* h, int64_t id, int32_t* out, int cap);
+int lt_sched_slot(void* h, int64_t id);
+int lt_sched_session_open(void* h, int64_t id);
+int lt_sched_session_grow(void* h, int64_t id, int n_tokens);
+int lt_sched_session_close(void* h, int64_t id);
 int lt_sched_context_len(void* h, int64_t id);
 int lt_sched_pop_finished(void* h, int64_t* ids, int cap);
 void lt_sched_release(void* h, int64_t id);

@@ -32,21 +32,28 @@ struct Req {
   int planned_chunk = 0;
   bool finished = false;
   std::vector<int32_t> blocks;
+  int slot = -1;                 // row of the per-sequence state arrays (recurrent layers) while the request is active
 };
 
 struct Sched {
   int num_blocks, block_size, max_seqs, max_tokens, eos_id;
   std::vector<int32_t> free_blocks;
+  std::vector<int32_t> free_slots;
   std::deque<std::shared_ptr<Req>> pending;
   std::vector<std::shared_ptr<Req>> running;
   std::vector<std::shared_ptr<Req>> done;
   std::unordered_map<int64_t, std::shared_ptr<Req>> by_id;
   std::mutex mu;
 
+  void give_back(Req& r) {
+    for (int32_t b : r.blocks) free_blocks.push_back(b);
+    r.blocks.clear();
+    if (r.slot >= 0) free_slots.push_back(r.slot);
+    r.slot = -1;
+  }
   void finish(const std::shared_ptr<Req>& r) {
     r->finished = true;
-    for (int32_t b : r->blocks) free_blocks.push_back(b);
-    r->blocks.clear();
+    give_back(*r);
     running.erase(std::remove(running.begin(), running.end(), r), running.end());
     done.push_back(r);
   }
@@ -82,6 +89,7 @@ void* lt_sched_create(int num_blocks, int block_size, int max_num_seqs, int max_
   s->num_blocks = num_blocks; s->block_size = block_size; s->max_seqs = max_num_seqs;
   s->max_tokens = max_num_batched_tokens; s->eos_id = eos_id;
   for (int i = num_blocks - 1; i >= 0; --i) s->free_blocks.push_back(i);
+  for (int i = max_num_seqs - 1; i >= 0; --i) s->free_slots.push_back(i);
   return s;
 }
 void lt_sched_destroy(void* h) { delete static_cast<Sched*>(h); }
@@ -104,7 +112,7 @@ int lt_sched_add_request(void* h, int64_t id, const int32_t* prompt, int prompt_
 int lt_sched_plan(void* h, int64_t* req_ids, int32_t* chunk_start, int32_t* chunk_len, int cap) {
   Sched* s = static_cast<Sched*>(h);
   std::lock_guard<std::mutex> lk(s->mu);
-  while (int(s->running.size()) < s->max_seqs && !s->pending.empty()) {
+  while (int(s->running.size()) < s->max_seqs && !s->free_slots.empty() && !s->pending.empty()) {
     auto r = s->pending.front();
     const size_t total = r->prompt.size() + size_t(r->max_new);
     const size_t need = (total + s->block_size - 1) / s->block_size;
@@ -114,6 +122,8 @@ int lt_sched_plan(void* h, int64_t* req_ids, int32_t* chunk_start, int32_t* chun
       r->blocks.push_back(s->free_blocks.back());
       s->free_blocks.pop_back();
     }
+    r->slot = s->free_slots.back();
+    s->free_slots.pop_back();
     s->running.push_back(r);
   }
   int budget = s->max_tokens;
@@ -180,6 +190,55 @@ int lt_sched_block_table(void* h, int64_t id, int32_t* out, int cap) {
   int n = 0;
   for (int32_t b : it->second->blocks) if (n < cap) out[n++] = b;
   return int(it->second->blocks.size());
+}
+
+// State slot of an active request or session, -1 otherwise.
+int lt_sched_slot(void* h, int64_t id) {
+  Sched* s = static_cast<Sched*>(h);
+  std::lock_guard<std::mutex> lk(s->mu);
+  auto it = s->by_id.find(id);
+  return it == s->by_id.end() ? -1 : it->second->slot;
+}
+
+// Sessions: sequences whose tokens the caller brings step by step.  They hold blocks and a slot of the same pools as
+// requests but are never planned.  Returns the slot, -1 for a known id, -2 when every slot is taken.
+int lt_sched_session_open(void* h, int64_t id) {
+  Sched* s = static_cast<Sched*>(h);
+  std::lock_guard<std::mutex> lk(s->mu);
+  if (s->by_id.count(id)) return -1;
+  if (s->free_slots.empty()) return -2;
+  auto r = std::make_shared<Req>();
+  r->id = id;
+  r->max_new = 0;
+  r->slot = s->free_slots.back();
+  s->free_slots.pop_back();
+  s->by_id[id] = r;
+  return r->slot;
+}
+// Blocks for the first n_tokens positions; returns how many the session now has, -1 when the pool is too small (nothing
+// is taken then).
+int lt_sched_session_grow(void* h, int64_t id, int n_tokens) {
+  Sched* s = static_cast<Sched*>(h);
+  std::lock_guard<std::mutex> lk(s->mu);
+  auto it = s->by_id.find(id);
+  if (it == s->by_id.end()) return -1;
+  auto& r = *it->second;
+  const size_t need = (size_t(n_tokens) + s->block_size - 1) / s->block_size;
+  if (need > r.blocks.size() + s->free_blocks.size()) return -1;
+  while (r.blocks.size() < need) {
+    r.blocks.push_back(s->free_blocks.back());
+    s->free_blocks.pop_back();
+  }
+  return int(r.blocks.size());
+}
+int lt_sched_session_close(void* h, int64_t id) {
+  Sched* s = static_cast<Sched*>(h);
+  std::lock_guard<std::mutex> lk(s->mu);
+  auto it = s->by_id.find(id);
+  if (it == s->by_id.end()) return -1;
+  s->give_back(*it->second);
+  s->by_id.erase(it);
+  return 0;
 }
 
 int lt_sched_context_len(void* h, int64_t id) {

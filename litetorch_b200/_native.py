@@ -15,7 +15,9 @@ ranks, the data-loader workers, tests without a GPU) never touch the CUDA runtim
 from __future__ import annotations
 
 import ctypes
+import fcntl
 import glob
+import hashlib
 import os
 import shutil
 import subprocess
@@ -59,16 +61,54 @@ def cuda_sources():
         glob.glob(os.path.join(_CSRC, "cuda_runtime", "*.cu")))
 
 
+# Sets of sources that a program which needs only a part of the library can build by themselves (`ensure_cuda`).
+COMPONENTS = {
+    "serving": ["common/host.cu", "gemm_sm100.cu", "gemm_skinny.cu", "gemv.cu", "flash_fwd.cu", "paged_decode.cu", "pointwise.cu"],
+    "hybrid": ["hyper_norm.cu", "gemm_simt.cu", "window_attn.cu", "rglru.cu", "mlstm.cu"],
+}
+
+
+def component_sources(components):
+    if "all" in components:
+        return cuda_sources()
+    return sorted(os.path.join(_CSRC, "kernels", f) for c in components for f in COMPONENTS[c])
+
+
+def _library_path(components) -> str:
+    return os.path.join(_LIB, "liblt_cuda.so" if "all" in components else "liblt_cuda_%s.so" % "_".join(sorted(components)))
+
+
+def _source_hash(components) -> str:
+    """Digest of everything a library of these components is made from."""
+    h = hashlib.sha256(" ".join(NVCC_FLAGS).encode())
+    hdrs = glob.glob(os.path.join(_CSRC, "**", "*.cuh"), recursive=True) + glob.glob(os.path.join(_CSRC, "**", "*.h"), recursive=True)
+    for f in sorted(hdrs) + component_sources(components):
+        h.update(os.path.relpath(f, _CSRC).encode())
+        with open(f, "rb") as fh:
+            h.update(fh.read())
+    return h.hexdigest()
+
+
+def _is_current(components) -> bool:
+    path = _library_path(components)
+    try:
+        with open(path + ".src") as f:
+            return os.path.exists(path) and f.read().strip() == _source_hash(components)
+    except OSError:
+        return False
+
+
 def host_sources():
     return sorted(glob.glob(os.path.join(_CSRC, "runtime", "*.cpp")))
 
 
-def build_cuda(force: bool = False, verbose: bool = False) -> str:
-    """Compile every .cu under csrc/ for sm_100a and link liblt_cuda.so (cross-compiles without a GPU)."""
+def build_cuda(force: bool = False, verbose: bool = False, components=("all",)) -> str:
+    """Compile every .cu under csrc/ (or those of some components) for sm_100a and link liblt_cuda.so (a library named after
+    the components); cross-compiles without a GPU."""
     os.makedirs(_LIB, exist_ok=True)
     os.makedirs(_OBJ, exist_ok=True)
-    out = os.path.join(_LIB, "liblt_cuda.so")
-    srcs = cuda_sources()
+    out = _library_path(components)
+    srcs = component_sources(components)
     hdrs = glob.glob(os.path.join(_CSRC, "**", "*.cuh"), recursive=True) + glob.glob(
         os.path.join(_CSRC, "**", "*.h"), recursive=True)
     hdr_time = _newest(hdrs)
@@ -89,6 +129,8 @@ def build_cuda(force: bool = False, verbose: bool = False) -> str:
         cmd = [nvcc, "-shared", "-o", out + ".tmp"] + objs + ["-ldl"]
         _compile_one(cmd, out)
         os.replace(out + ".tmp", out)      # a reader never sees a half-written library
+    with open(out + ".src", "w") as f:
+        f.write(_source_hash(components))
     return out
 
 
@@ -159,6 +201,26 @@ def host_lib() -> ctypes.CDLL:
                 build_host()
             _host = ctypes.CDLL(path, mode=ctypes.RTLD_GLOBAL)
     return _host
+
+
+def ensure_cuda(components=("all",)) -> ctypes.CDLL:
+    """The native library with at least these components, for a program that starts from a source checkout: the whole
+    library where it is built and up to date, otherwise the components alone, compiled now if need be."""
+    global _cuda
+    if _cuda is not None:
+        return _cuda
+    if _is_current(("all",)):
+        return cuda_lib()
+    if not _is_current(components):
+        os.makedirs(_LIB, exist_ok=True)
+        with open(os.path.join(_LIB, ".build.lock"), "w") as lock:      # two programs that start together build once
+            fcntl.flock(lock, fcntl.LOCK_EX)
+            if not _is_current(components):
+                build_cuda(components=components)
+    with _lock:
+        if _cuda is None:
+            _cuda = ctypes.CDLL(_library_path(components), mode=ctypes.RTLD_GLOBAL)
+    return _cuda
 
 
 def have_cuda_lib() -> bool:

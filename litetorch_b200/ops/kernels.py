@@ -16,6 +16,23 @@ from .._native import cuda_lib
 _vp, _i, _ll, _f = c_void_p, c_int, c_longlong, c_float
 
 _SIGS = {
+    "lt_flash_fwd_window": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _ll, _ll, _ll, _ll, _ll, _ll, _ll, _ll, _f, _i, _vp],
+    "lt_paged_decode_window": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _f, _i, _vp, _ll, _i, _vp],
+    "lt_clamped_glu": [_i, _vp, _vp, _ll, _i, _f, _f, _vp],
+    "lt_gemm_block_diag": [_vp, _vp, _vp, _i, _i, _i, _i, _ll, _ll, _vp],
+    "lt_hyper_norm": [_i, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _f, _vp, _ll, _vp, _i, _i, _i, _i, _vp],
+    "lt_gemm_simt": [_i, _i, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _i, _ll, _ll, _ll, _f, _vp],
+    "lt_rows_dot": [_i, _vp, _ll, _vp, _vp, _i, _i, _i, _vp],
+    "lt_qkv_rope": [_i, _vp, _ll] + [_i] * 10 + [_vp, _vp, _f, _vp, _vp, _vp, _i, _f, _vp, _vp, _vp, _i, _vp, _vp, _vp],
+    "lt_kv_gather": [_vp, _vp, _vp, _vp, _vp] + [_i] * 6 + [_vp],
+    "lt_window_attn": [_i, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _ll] + [_i] * 9 + [_f, _vp],
+    "lt_head_gate": [_i, _vp, _vp, _ll, _vp, _ll, _i, _i, _i, _vp],
+    "lt_conv_causal": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "lt_rglru_scan": [_i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "lt_rglru_step": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "lt_mlstm_prefill": [_vp, _vp, _vp, _ll, _vp, _vp, _vp, _f, _f, _vp, _f, _vp, _ll] + [_vp] * 11 + [_i] * 5 + [_vp],
+    "lt_mlstm_step": [_i, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _vp, _vp] + [_i] * 7 + [_vp],
+    "lt_head_norm_gate": [_i, _vp, _vp, _vp, _ll, _vp, _ll, _i, _i, _f, _vp],
     "lt_status_fetch": [],
     "lt_sm_count": [],
     "lt_set_wait_budget_cycles": [_ll, _ll],
@@ -92,7 +109,7 @@ _SIGS = {
 _bound = {}
 
 # Kernels launched per native call; `launch_count()` is what bench.py reports as "gpu_launches".
-_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
+_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_paged_decode_window": 2, "lt_mlstm_prefill": 4, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
                       "lt_adam_chunk_elems": 0}
 _launches = [0]
 
@@ -113,7 +130,10 @@ def _fn(name):
     f = _bound.get(name)
     if f is None:
         lib = cuda_lib()
-        raw = getattr(lib, name)
+        try:
+            raw = getattr(lib, name)
+        except AttributeError:
+            raise KernelError("%s is not in the native library that is loaded (a partial or an old build)" % name) from None
         raw.argtypes = _SIGS[name]
         raw.restype = c_int
         n = _LAUNCHES_PER_CALL.get(name, 1)
@@ -445,6 +465,14 @@ def swiglu_fwd(gu: torch.Tensor) -> torch.Tensor:
     return h
 
 
+def clamped_glu(gu: torch.Tensor, limit: float, slope: float = 1.702) -> torch.Tensor:
+    """g sigmoid(slope g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); gu is [M, gate | up]."""
+    M, F2 = gu.shape
+    h = torch.empty((M, F2 // 2), dtype=gu.dtype, device=gu.device)
+    _check(_fn("lt_clamped_glu")(_f32(gu), gu.data_ptr(), h.data_ptr(), M, F2 // 2, float(limit), float(slope), _stream()), "lt_clamped_glu")
+    return h
+
+
 def swiglu_bwd(gu: torch.Tensor, dh: torch.Tensor, inplace: bool = True) -> torch.Tensor:
     M, F2 = gu.shape
     dgu = gu if inplace else torch.empty_like(gu)
@@ -551,13 +579,21 @@ def clip_coef(stats: torch.Tensor, dyn: torch.Tensor, max_norm: float, inv_scale
 
 
 # ------------------------------------------------------------------------------------------------ attention
-def flash_fwd(q, k, v, *, causal=True, scale=None):
-    """q: [B, Tq, Hq, D], k/v: [B, Tk, Hkv, D] (last dim contiguous, arbitrary other strides).  Returns (o, lse)."""
+def flash_fwd(q, k, v, *, causal=True, scale=None, window=0):
+    """q: [B, Tq, Hq, D], k/v: [B, Tk, Hkv, D] (last dim contiguous, arbitrary other strides).  Returns (o, lse).
+    window > 0 (causal only): a query sees its own position and the window - 1 before it."""
     B, Tq, Hq, D = q.shape
     _, Tk, Hkv, _ = k.shape
     scale = (D ** -0.5) if scale is None else scale
     o = torch.empty((B, Tq, Hq, D), dtype=q.dtype, device=q.device)
     lse = torch.empty((B, Hq, Tq), dtype=torch.float32, device=q.device)
+    if window > 0:
+        assert causal
+        rc = _fn("lt_flash_fwd_window")(q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), lse.data_ptr(), B, Tq, Tk, Hq, Hkv, D,
+                                        q.stride(0), q.stride(1), k.stride(0), k.stride(1), v.stride(0), v.stride(1),
+                                        o.stride(0), o.stride(1), float(scale), int(window), _stream())
+        _check(rc, "lt_flash_fwd_window")
+        return o, lse
     rc = _fn("lt_flash_fwd")(q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), lse.data_ptr(), B, Tq, Tk, Hq, Hkv, D,
                              q.stride(0), q.stride(1), k.stride(0), k.stride(1), v.stride(0), v.stride(1),
                              o.stride(0), o.stride(1), float(scale), 1 if causal else 0, _stream())
@@ -682,17 +718,21 @@ def signal_barrier(my_flags, peer_flag_ptrs, slot: int, epoch: int, world: int, 
 
 # ------------------------------------------------------------------------------------------------ serving
 def paged_decode(q, k_cache, v_cache, block_tables, context_lens, block_size: int, splits: int, scale: float,
-                 k_scale: float = 1.0, v_scale: float = 1.0):
+                 k_scale: float = 1.0, v_scale: float = 1.0, window: int = 0, gate=None, vdim: int = 0):
+    """Attention of q [S, H, D] over paged caches.  window > 0: the newest `window` keys of every sequence; gate: logits
+    [S, H] (rows may be strided), every head's output is multiplied by the sigmoid of its own; vdim: how many of the D
+    value columns are meant (0: all) - the result is [S, H, vdim]."""
     S, H, D = q.shape
     Hkv = k_cache.shape[1]
     part = torch.empty((S, H, splits, D + 2), dtype=torch.float32, device=q.device)
-    o = torch.empty_like(q)
-    rc = _fn("lt_paged_decode")(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr(),
-                                context_lens.data_ptr(), part.data_ptr(), o.data_ptr(), S, H, Hkv, D, block_size,
-                                block_tables.shape[1], k_cache.shape[0] if k_cache.is_contiguous() and v_cache.is_contiguous() else 0, splits,
-                                float(scale), 1 if k_cache.dtype == torch.float8_e4m3fn else 0,
-                                float(k_scale), float(v_scale), _stream())
-    _check(rc, "lt_paged_decode")
+    vdim = vdim or D
+    o = torch.empty((S, H, vdim), dtype=q.dtype, device=q.device)
+    rc = _fn("lt_paged_decode_window")(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr(),
+                                       context_lens.data_ptr(), part.data_ptr(), o.data_ptr(), S, H, Hkv, D, block_size,
+                                       block_tables.shape[1], k_cache.shape[0] if k_cache.is_contiguous() and v_cache.is_contiguous() else 0, splits,
+                                       float(scale), 1 if k_cache.dtype == torch.float8_e4m3fn else 0, float(k_scale), float(v_scale),
+                                       int(window), _p(gate), gate.stride(0) if gate is not None else 0, vdim, _stream())
+    _check(rc, "lt_paged_decode_window")
     return o
 
 
@@ -751,6 +791,210 @@ def flash_bwd_cp(phase, *, q_ptrs, k, v, o, do_ptrs, lse_ptrs, delta_ptrs, dq_ac
                                 q_like.stride(1), q_like.stride(0), q_like.stride(1), k.stride(0), k.stride(1), float(scale),
                                 1 if causal else 0, cp_world, cp_rank, 1 if zigzag else 0, _stream())
     _check(rc, "lt_flash_bwd_cp")
+
+
+# ------------------------------------------------------------------------------------------------ hybrid decoders
+# Everything below runs on bf16 or fp32 activations (the dtype of the tensors decides); fp32 is true fp32.
+def _f32(t) -> int:
+    if t.dtype == torch.float32:
+        return 1
+    assert t.dtype == torch.bfloat16, t.dtype
+    return 0
+
+
+def linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None, alpha: float = 1.0) -> torch.Tensor:
+    """alpha * x[M, K] @ w[N, K]^T.  bf16 goes to the tensor-core GEMMs of `gemm`; fp32, and bf16 operands that TMA cannot
+    describe (K or a pitch not a multiple of 8), to the CUDA-core kernel."""
+    out_dtype = out_dtype or x.dtype
+    assert x.stride(1) == 1 and w.is_contiguous() and x.dtype == w.dtype and x.shape[1] == w.shape[1]
+    (M, Kd), N = x.shape, w.shape[0]
+    if M == 0:
+        return torch.empty((0, N), dtype=out_dtype, device=x.device)
+    if x.dtype == torch.bfloat16 and Kd % 8 == 0 and (M == 1 or x.stride(0) % 8 == 0) and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
+        return gemm(x, w, out_dtype=out_dtype, alpha=alpha)
+    y = torch.empty((M, N), dtype=out_dtype, device=x.device)
+    rc = _fn("lt_gemm_simt")(_f32(x), _f32(y), x.data_ptr(), w.data_ptr(), y.data_ptr(), M, N, Kd, x.stride(0), Kd, N, 1, 0, 0, 0,
+                             float(alpha), _stream())
+    _check(rc, "lt_gemm_simt")
+    return y
+
+
+def block_diag(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x [M, B * K] times the block-diagonal matrix w [B, N, K]: fp32 [M, B * N] with columns z N .. from block z."""
+    B, N, Kd = w.shape
+    M = x.shape[0]
+    assert x.shape[1] == B * Kd and x.is_contiguous() and w.is_contiguous() and x.dtype == w.dtype
+    y = torch.empty((M, B * N), dtype=torch.float32, device=x.device)
+    if x.dtype == torch.bfloat16 and Kd % 8 == 0 and N % 128 == 0:
+        rc = _fn("lt_gemm_block_diag")(x.data_ptr(), w.data_ptr(), y.data_ptr(), M, B, N, Kd, x.stride(0), y.stride(0), _stream())
+        _check(rc, "lt_gemm_block_diag")
+        return y
+    rc = _fn("lt_gemm_simt")(_f32(x), 1, x.data_ptr(), w.data_ptr(), y.data_ptr(), M, N, Kd, B * Kd, Kd, B * N, B, Kd, N * Kd, N, 1.0, _stream())
+    _check(rc, "lt_gemm_simt")
+    return y
+
+
+def rows_dot(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x[R, K] @ w[J, K]^T as fp32 [R, J] for a narrow w (gates of a recurrence: their logits stay fp32)."""
+    assert x.stride(1) == 1 and w.is_contiguous() and x.dtype == w.dtype
+    y = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
+    rc = _fn("lt_rows_dot")(_f32(x), x.data_ptr(), x.stride(0), w.data_ptr(), y.data_ptr(), x.shape[0], w.shape[0], x.shape[1], _stream())
+    _check(rc, "lt_rows_dot")
+    return y
+
+
+def hyper_norm(x, norm, eps: float, *, dtype, inn=None, tokens=None, embed=None, y=None, y_norm=None, y2=None, y2_norm=None,
+               mix=None, out=None, rows=None, write=True):
+    """One step along the residual streams x [T, streams, W] (fp32, updated in place): add the finished sublayer's output y
+    (x_t <- sum_s mix[s, t] x_s + out[t] y; with y2, the half sum of y and y2 normed with y_norm / y2_norm), then return
+    the RMS norm of sum_s inn[s] x_s (inn None: the plain sum) as [rows, W] of `dtype`.  With `embed` the streams start as
+    embed[tokens]; `rows` picks tokens; write=False leaves x alone."""
+    T, S, W = x.shape
+    n = T if rows is None else rows.shape[0]
+    h = torch.empty((n, W), dtype=dtype, device=x.device)
+    if n == 0:
+        return h
+    assert x.is_contiguous() and x.dtype == torch.float32 and (y is None or y.dtype == dtype) and (embed is None or embed.dtype == dtype)
+    rc = _fn("lt_hyper_norm")(_f32(h), x.data_ptr(), _p(tokens), _p(embed), _p(y), y.stride(0) if y is not None else 0, _p(y_norm),
+                              _p(y2), y2.stride(0) if y2 is not None else 0, _p(y2_norm), _p(mix), _p(out), _p(inn), norm.data_ptr(),
+                              float(eps), h.data_ptr(), h.stride(0), _p(rows), n, W, S, 1 if write else 0, _stream())
+    _check(rc, "lt_hyper_norm")
+    return h
+
+
+def qkv_rope(proj, q_off: int, k_off: int, v_off: int, H: int, G: int, D: int, E: int, positions, slots, k_cache, v_cache, *,
+             freq, rot_dims: int, gain: float = 1.0, q_norm=None, k_norm=None, eps: float = 1e-6, lin=None):
+    """Takes q, k and v out of the fused projection, norms q and k over the whole projection, rotates them (interleaved
+    pairs of the first rot_dims dimensions, angle position * freq[i], cos and sin times gain), writes k and v into the
+    paged caches (and, with lin = (k_lin, v_lin), one after another as well) and returns q [N, H, padded size]."""
+    N = proj.shape[0]
+    bs, DP, EP = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    q = torch.empty((N, H, DP), dtype=proj.dtype, device=proj.device)
+    k_lin, v_lin = lin if lin is not None else (None, None)
+    rc = _fn("lt_qkv_rope")(_f32(proj), proj.data_ptr(), proj.stride(0), N, q_off, k_off, v_off, H, G, D, E, DP, EP, _p(q_norm), _p(k_norm),
+                            float(eps), positions.data_ptr(), slots.data_ptr(), freq.data_ptr(), rot_dims, float(gain), q.data_ptr(),
+                            k_cache.data_ptr(), v_cache.data_ptr(), bs, _p(k_lin), _p(v_lin), _stream())
+    _check(rc, "lt_qkv_rope")
+    return q
+
+
+def kv_gather(k_cache, v_cache, table, pos0: int, n: int, k_lin, v_lin):
+    """Keys and values of positions pos0 .. pos0 + n - 1 of the sequence with block table `table` into k_lin / v_lin [n, G, .]."""
+    rc = _fn("lt_kv_gather")(k_cache.data_ptr(), v_cache.data_ptr(), k_lin.data_ptr(), v_lin.data_ptr(), table.data_ptr(), pos0, n,
+                             k_cache.shape[1], k_cache.shape[3] * k_cache.element_size(), v_cache.shape[3] * v_cache.element_size(),
+                             k_cache.shape[2], _stream())
+    _check(rc, "lt_kv_gather")
+
+
+def window_attn(q, k_cache, v_cache, tables, positions, *, D: int, E: int, window: int, scale: float, gate=None):
+    """CUDA-core attention of q [N, H, padded] over paged caches: row n attends to positions max(0, p - window + 1) .. p of
+    the sequence in tables[n] (tables 1-D: every row is of that one sequence).  Returns [N, H, E], gated as in `paged_decode`."""
+    N, H, DP = q.shape
+    o = torch.empty((N, H, E), dtype=q.dtype, device=q.device)
+    rc = _fn("lt_window_attn")(_f32(q), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), tables.data_ptr(),
+                               tables.stride(0) if tables.dim() == 2 else 0, positions.data_ptr(), o.data_ptr(), _p(gate),
+                               gate.stride(0) if gate is not None else 0, N, H, k_cache.shape[1], D, E, DP, v_cache.shape[3],
+                               k_cache.shape[2], int(window), float(scale), _stream())
+    _check(rc, "lt_window_attn")
+    return o
+
+
+def head_gate(o, gate, E: int):
+    """o [N, H, >= E] times sigmoid(gate [N, H]), packed to [N, H, E]."""
+    N, H, EP = o.shape
+    out = torch.empty((N, H, E), dtype=o.dtype, device=o.device)
+    rc = _fn("lt_head_gate")(_f32(o), o.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), N, H, E, EP, _stream())
+    _check(rc, "lt_head_gate")
+    return out
+
+
+def conv_causal(x, xb, w, b, ring, start: int):
+    """Causal convolution per channel of x [N, C] (+ bias xb), w [C, taps], at positions start ..; earlier inputs come from
+    `ring` [taps, C] (input of position p in row p % taps)."""
+    N, C = x.shape
+    u = torch.empty((N, C), dtype=x.dtype, device=x.device)
+    rc = _fn("lt_conv_causal")(_f32(x), x.data_ptr(), x.stride(0), _p(xb), w.data_ptr(), b.data_ptr(), ring.data_ptr(), u.data_ptr(), N, C,
+                               w.shape[1], start, _stream())
+    _check(rc, "lt_conv_causal")
+    return u
+
+
+def rglru_scan(u, gates, rb, ib, sp, y, yb, x, xb, state, ring, taps: int, start: int):
+    """The recurrence over a prompt chunk: u [N, C], gates fp32 [N, 2 C] (per block: logits of r, then of i), sp =
+    softplus(lam), y [N, C] the other branch; state [C] and ring [taps, C] are updated.  Returns S * gelu(y + yb)."""
+    N, C = u.shape
+    bw = rb.shape[-1]
+    out = torch.empty((N, C), dtype=u.dtype, device=u.device)
+    rc = _fn("lt_rglru_scan")(_f32(u), u.data_ptr(), gates.data_ptr(), rb.data_ptr(), ib.data_ptr(), sp.data_ptr(), y.data_ptr(), y.stride(0),
+                              yb.data_ptr(), x.data_ptr(), x.stride(0), _p(xb), state.data_ptr(), ring.data_ptr(), out.data_ptr(), N, C, bw,
+                              taps, start, _stream())
+    _check(rc, "lt_rglru_scan")
+    return out
+
+
+def rglru_step(x, xb, conv_w, conv_b, gates, rb, ib, sp, y, yb, state, ring, slots, positions):
+    """One token of every sequence: convolution, gates ([blocks, rows of r | rows of i, bw]), recurrence and output branch; row s uses
+    state[slots[s]] [C] and ring[slots[s]] [taps, C]."""
+    S, C = x.shape
+    out = torch.empty((S, C), dtype=x.dtype, device=x.device)
+    rc = _fn("lt_rglru_step")(_f32(x), x.data_ptr(), x.stride(0), _p(xb), conv_w.data_ptr(), conv_b.data_ptr(), gates.data_ptr(),
+                              rb.data_ptr(), ib.data_ptr(), sp.data_ptr(), y.data_ptr(), y.stride(0), yb.data_ptr(), state.data_ptr(),
+                              ring.data_ptr(), slots.data_ptr(), positions.data_ptr(), out.data_ptr(), S, C, rb.shape[-1], conv_w.shape[1],
+                              _stream())
+    _check(rc, "lt_rglru_step")
+    return out
+
+
+def mlstm_prefill(q, k, v, logits, ib, fb, cap: float, norm, eps: float, gate, S, n, m, D: int, E: int, start: int):
+    """A prompt chunk of one sequence through the matrix memory; q, k [N, H D], v [N, H E] (columns of one projection),
+    logits fp32 [N, 2 H], S [H, D, E], n [2, H, D], m [2, H] of its slot, updated.  Returns the normed and gated [N, H E]."""
+    N, H = q.shape[0], S.shape[0]
+    dev, f32 = q.device, torch.float32
+    assert q.stride(0) == k.stride(0) == v.stride(0)
+    qscale = D ** -0.5
+    if q.dtype == torch.float32:
+        o = torch.empty((N, H * E), dtype=f32, device=dev)
+        rc = _fn("lt_mlstm_step")(1, q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), logits.data_ptr(), ib.data_ptr(), fb.data_ptr(),
+                                  float(cap), qscale, S.data_ptr(), n.data_ptr(), m.data_ptr(), None, None, o.data_ptr(), 0, H, D, E, N, 0,
+                                  start, _stream())
+        _check(rc, "lt_mlstm_step")
+        return head_norm_gate(o, norm, gate, H, eps)
+    chunks = (N + 127) // 128
+    sizes = [H * N, H * N, H * N, H * (chunks + 1), H * chunks * D * E, H * chunks * D, N * H * E]
+    offs, total = [], 0
+    for s in sizes:
+        offs.append(total)
+        total += (s + 63) // 64 * 64
+    scratch = torch.empty(total, dtype=f32, device=dev)
+    base = scratch.data_ptr()
+    out = torch.empty((N, H * E), dtype=q.dtype, device=dev)
+    rc = _fn("lt_mlstm_prefill")(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), logits.data_ptr(), ib.data_ptr(), fb.data_ptr(),
+                                 float(cap), qscale, norm.data_ptr(), float(eps), gate.data_ptr(), gate.stride(0), S.data_ptr(), n.data_ptr(),
+                                 m.data_ptr(), *[base + 4 * o for o in offs], out.data_ptr(), N, H, D, E, start, _stream())
+    _check(rc, "lt_mlstm_prefill")
+    return out
+
+
+def mlstm_step(q, k, v, logits, ib, fb, cap: float, norm, eps: float, gate, S, n, m, slots, positions, D: int, E: int):
+    """One token of every sequence; S [slots, H, D, E], n [slots, 2, H, D], m [slots, 2, H]."""
+    R, H = q.shape[0], S.shape[1]
+    assert q.stride(0) == k.stride(0) == v.stride(0)
+    o = torch.empty((R, H * E), dtype=torch.float32, device=q.device)
+    rc = _fn("lt_mlstm_step")(_f32(q), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), logits.data_ptr(), ib.data_ptr(), fb.data_ptr(),
+                              float(cap), D ** -0.5, S.data_ptr(), n.data_ptr(), m.data_ptr(), slots.data_ptr(), positions.data_ptr(),
+                              o.data_ptr(), R, H, D, E, 0, 0, 0, _stream())
+    _check(rc, "lt_mlstm_step")
+    return head_norm_gate(o, norm, gate, H, eps)
+
+
+def head_norm_gate(o, w, gate, H: int, eps: float):
+    """RMS norm per head of o (fp32 [R, H E]), times w [H E] and sigmoid(gate [R, H E]), in the gate's dtype."""
+    R, HE = o.shape
+    out = torch.empty((R, HE), dtype=gate.dtype, device=o.device)
+    rc = _fn("lt_head_norm_gate")(_f32(out), o.data_ptr(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), R, H, HE // H,
+                                  float(eps), _stream())
+    _check(rc, "lt_head_norm_gate")
+    return out
 
 
 # ------------------------------------------------------------------------------------------------ mixture of experts

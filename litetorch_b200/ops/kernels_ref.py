@@ -184,7 +184,7 @@ def _expand_kv(k, Hq):
     return k if Hkv == Hq else k[:, :, :, None, :].expand(B, T, Hkv, Hq // Hkv, D).reshape(B, T, Hq, D)
 
 
-def flash_fwd(q, k, v, *, causal=True, scale=None):
+def flash_fwd(q, k, v, *, causal=True, scale=None, window=0):
     B, Tq, Hq, D = q.shape
     Tk = k.shape[1]
     scale = (D ** -0.5) if scale is None else scale
@@ -194,6 +194,8 @@ def flash_fwd(q, k, v, *, causal=True, scale=None):
     s = qf @ kf.transpose(-1, -2) * scale
     if causal:
         mask = torch.ones(Tq, Tk, dtype=torch.bool, device=q.device).tril(Tk - Tq)
+        if window > 0:
+            mask = mask.triu(Tk - Tq - window + 1)
         s = s.masked_fill(~mask, float("-inf"))
     lse = torch.logsumexp(s, -1)
     o = torch.exp(s - lse[..., None]) @ vf
@@ -266,3 +268,179 @@ def clip_coef(stats, dyn, max_norm, inv_scale=1.0):
     dyn[1] = 1.0 if float(stats[1]) != 0.0 else 0.0
     dyn[2] = norm
     return dyn
+
+
+# ------------------------------------------------------------------------------------------------ hybrid decoders
+def clamped_glu(gu, limit, slope=1.702):
+    g, u = gu.float().chunk(2, -1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(slope * g) * (u + 1)).to(gu.dtype)
+
+
+def linear(x, w, out_dtype=None, alpha=1.0):
+    return (x.float() @ w.float().t() * alpha).to(out_dtype or x.dtype)
+
+
+def block_diag(x, w):
+    B, N, Kd = w.shape
+    return torch.matmul(x.float().view(-1, B, 1, Kd), w.float().transpose(1, 2)).reshape(x.shape[0], B * N)
+
+
+def rows_dot(x, w):
+    return x.float() @ w.float().t()
+
+
+def _rms(x, eps, w=None):
+    y = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+    return y if w is None else y * w
+
+
+def hyper_norm(x, norm, eps, *, dtype, inn=None, tokens=None, embed=None, y=None, y_norm=None, y2=None, y2_norm=None, mix=None,
+               out=None, rows=None, write=True):
+    xs = x if embed is None else embed[tokens.long()].float()[:, None].expand(x.shape)
+    if y is not None:
+        y = y.float() if y2 is None else 0.5 * (_rms(y.float(), eps, y_norm) + _rms(y2.float(), eps, y2_norm))
+    if rows is not None:
+        xs = xs[rows.long()]
+        y = None if y is None else y[rows.long()]
+    if y is not None:
+        xs = torch.matmul(mix.t(), xs) + out[:, None] * y[:, None]
+    if write:
+        x.copy_(xs)
+    u = xs.sum(1) if inn is None else torch.matmul(inn, xs)
+    return _rms(u, eps, norm).to(dtype)
+
+
+def qkv_rope(proj, q_off, k_off, v_off, H, G, D, E, positions, slots, k_cache, v_cache, *, freq, rot_dims, gain=1.0, q_norm=None,
+             k_norm=None, eps=1e-6, lin=None):
+    N = proj.shape[0]
+    bs, DP, EP = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    angle = positions.double()[:, None] * freq[None]
+    c, s = (torch.cos(angle) * gain).float()[:, None], (torch.sin(angle) * gain).float()[:, None]
+
+    def take(off, heads, w):
+        t = proj[:, off:off + heads * D].float()
+        t = (t if w is None else _rms(t, eps, w)).reshape(N, heads, D).clone()
+        u, v = t[..., 0:rot_dims:2].clone(), t[..., 1:rot_dims:2].clone()
+        t[..., 0:rot_dims:2], t[..., 1:rot_dims:2] = u * c - v * s, v * c + u * s
+        return torch.nn.functional.pad(t, (0, DP - D)).to(proj.dtype)
+
+    q, k = take(q_off, H, q_norm), take(k_off, G, k_norm)
+    v = torch.nn.functional.pad(proj[:, v_off:v_off + G * E].reshape(N, G, E), (0, EP - E))
+    blk, off = slots.long() // bs, slots.long() % bs
+    k_cache[blk, :, off] = k
+    v_cache[blk, :, off] = v
+    if lin is not None:
+        lin[0].copy_(k)
+        lin[1].copy_(v)
+    return q
+
+
+def kv_gather(k_cache, v_cache, table, pos0, n, k_lin, v_lin):
+    p = torch.arange(pos0, pos0 + n)
+    blk, off = table.long()[p // k_cache.shape[2]], p % k_cache.shape[2]
+    k_lin.copy_(k_cache[blk, :, off])
+    v_lin.copy_(v_cache[blk, :, off])
+
+
+def window_attn(q, k_cache, v_cache, tables, positions, *, D, E, window, scale, gate=None):
+    N, H, _ = q.shape
+    G, bs = k_cache.shape[1], k_cache.shape[2]
+    o = torch.empty(N, H, E, dtype=torch.float32)
+    for i in range(N):
+        pos = int(positions[i])
+        p = torch.arange(max(0, pos - window + 1) if window > 0 else 0, pos + 1)
+        t = tables if tables.dim() == 1 else tables[i]
+        blk = t.long()[p // bs]
+        k = k_cache[blk, :, p % bs][..., :D].float().repeat_interleave(H // G, 1)
+        v = v_cache[blk, :, p % bs][..., :E].float().repeat_interleave(H // G, 1)
+        w = torch.softmax(torch.einsum("hd,jhd->hj", q[i, :, :D].float(), k) * scale, -1)
+        o[i] = torch.einsum("hj,jhe->he", w, v)
+    if gate is not None:
+        o = o * torch.sigmoid(gate.float())[..., None]
+    return o.to(q.dtype)
+
+
+def head_gate(o, gate, E):
+    return (o[..., :E].float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
+
+
+def conv_causal(x, xb, w, b, ring, start):
+    N, C = x.shape
+    taps = w.shape[1]
+    xin = x.float() if xb is None else x.float() + xb
+    head = torch.zeros(taps - 1, C)
+    for k in range(taps - 1):
+        pos = start - (taps - 1) + k
+        if pos >= 0:
+            head[k] = ring[pos % taps]
+    full = torch.cat([head, xin])
+    return (sum(full[k:k + N] * w[:, k] for k in range(taps)) + b).to(x.dtype)
+
+
+def _rglru_coefficients(r, i, u, sp):
+    log_a = -8.0 * torch.sigmoid(r) * sp
+    return torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * torch.sigmoid(i) * u.float()
+
+
+def rglru_scan(u, gates, rb, ib, sp, y, yb, x, xb, state, ring, taps, start):
+    N, C = u.shape
+    B, bw = rb.shape
+    g = gates.view(N, B, 2, bw)
+    a, b = _rglru_coefficients((g[:, :, 0] + rb).reshape(N, C), (g[:, :, 1] + ib).reshape(N, C), u, sp)
+    s = state.clone() if start > 0 else torch.zeros(C)
+    out = torch.empty(N, C)
+    for t in range(N):
+        s = a[t] * s + b[t]
+        out[t] = s
+    state.copy_(s)
+    for t in range(max(0, N - taps), N):
+        ring[(start + t) % taps] = x[t].float() + (0 if xb is None else xb)
+    return (out * torch.nn.functional.gelu(y.float() + yb, approximate="tanh")).to(u.dtype)
+
+
+def rglru_step(x, xb, conv_w, conv_b, gates, rb, ib, sp, y, yb, state, ring, slots, positions):
+    rows = []
+    for s in range(x.shape[0]):
+        slot, pos = int(slots[s]), int(positions[s])
+        u = conv_causal(x[s:s + 1], xb, conv_w, conv_b, ring[slot], pos)
+        rows.append(rglru_scan(u, block_diag(u, gates), rb, ib, sp, y[s:s + 1], yb, x[s:s + 1], xb, state[slot], ring[slot], conv_w.shape[1], pos))
+    return torch.cat(rows)
+
+
+def mlstm_prefill(q, k, v, logits, ib, fb, cap, norm, eps, gate, S, n, m, D, E, start):
+    N, H = q.shape[0], S.shape[0]
+    i = cap * torch.tanh((logits[:, :H] + ib) / cap)
+    f = torch.nn.functional.logsigmoid(cap * torch.tanh((logits[:, H:] + fb) / cap))
+    qf, kf, vf = q.reshape(N, H, D).float() * D ** -0.5, k.reshape(N, H, D).float(), v.reshape(N, H, E).float()
+    bank = start & 1
+    Sc, nc, mc = (S.clone(), n[bank].clone(), m[bank].clone()) if start > 0 else (torch.zeros_like(S), torch.zeros(H, D), torch.zeros(H))
+    o = torch.empty(N, H, E)
+    for t in range(N):
+        m1 = torch.maximum(f[t] + mc, i[t])
+        keep, add = torch.exp(f[t] + mc - m1), torch.exp(i[t] - m1)
+        Sc = keep[:, None, None] * Sc + (add[:, None] * kf[t])[:, :, None] * vf[t][:, None, :]
+        nc = keep[:, None] * nc + add[:, None] * kf[t]
+        mc = m1
+        den = torch.maximum((nc * qf[t]).sum(-1).abs(), torch.exp(-mc)) + 1e-6
+        o[t] = torch.einsum("hd,hde->he", qf[t], Sc) / den[:, None]
+    bank = (start + N) & 1
+    S.copy_(Sc)
+    n[bank].copy_(nc)
+    m[bank].copy_(mc)
+    return head_norm_gate(o.view(N, H * E), norm, gate, H, eps)
+
+
+def mlstm_step(q, k, v, logits, ib, fb, cap, norm, eps, gate, S, n, m, slots, positions, D, E):
+    rows = []
+    for s in range(q.shape[0]):
+        j = slice(s, s + 1)
+        slot = int(slots[s])
+        rows.append(mlstm_prefill(q[j], k[j], v[j], logits[j], ib, fb, cap, norm, eps, gate[j], S[slot], n[slot], m[slot], D, E, int(positions[s])))
+    return torch.cat(rows)
+
+
+def head_norm_gate(o, w, gate, H, eps):
+    R, HE = o.shape
+    y = _rms(o.view(R, H, HE // H), eps).reshape(R, HE) * w
+    return (y * torch.sigmoid(gate.float())).to(gate.dtype)
