@@ -18,19 +18,16 @@ import torch
 
 from ..serving import PagedKVCache
 from .llama import LlamaEngine
+from .serving_base import Sampler, ServingModel, generate          # noqa: F401  (their names live here as well)
 
 
-class LlamaKVModel:
+class LlamaKVModel(ServingModel):
     def __init__(self, engine: LlamaEngine, num_blocks: int, block_size: int = 16, kv_dtype=torch.bfloat16, num_splits: int = 0,
                  graphs: bool = True, prefix_cache_bytes: int = 0):
         assert engine.w.tp == 1 and hasattr(engine.w, "flat_p"), "serving runs on whole (unsharded) weights"
-        self.e = engine
+        super().__init__(engine, block_size, graphs)
         cfg = engine.cfg
-        self.block_size = block_size
         self.num_splits = num_splits
-        self.graphs = graphs                 # record the decode step per (batch size, table width) and replay it
-        self._graphs = {}
-        self.sampler = None                  # None: greedy on the device; else a callable logits [rows, vocab] -> tokens
         self.cache = PagedKVCache(cfg.n_layers, num_blocks, block_size, cfg.n_kv_heads, cfg.head_dim, device=engine.device,
                                   dtype=kv_dtype)
         self.kv_bytes_per_token = 2 * cfg.n_layers * cfg.n_kv_heads * cfg.head_dim * self.cache.k[0].element_size()
@@ -39,8 +36,6 @@ class LlamaKVModel:
         # and only its remaining tokens are computed.  The reference has the prefix map (src/llm/prefix_cache.cpp) but
         # never consults it while serving.
         self.prefix_cache_bytes = int(prefix_cache_bytes)
-        self.prefill_tokens_computed = 0
-        self.prefill_tokens_reused = 0
         self._snap = OrderedDict()           # handle -> (k [layers, nb, Hkv, bs, hd], v, bytes)
         self._snap_bytes = 0
         self._next_handle = 1
@@ -70,28 +65,20 @@ class LlamaKVModel:
             x = K.gemm(hm, w.p(p + "w_down"), residual=x1)
         return x
 
-    def _next_tokens(self, x_rows):
+    def _logits(self, hidden, rows=None):
         e, K = self.e, self.e.K
-        hf, _, _, _ = K.norm_fwd(x_rows, e.w.p("final_norm"), eps=e.cfg.rms_eps)
-        logits = K.gemm(hf, e.w.p("lm_head"))
-        self.last_logits = logits            # [rows, vocab] of the newest step (kept for inspection and tests)
-        if self.sampler is not None:
-            return self.sampler(logits.float())
-        return logits.float().argmax(-1)
-
-    def _slots(self, block_ids: Sequence[int], start: int, n: int) -> torch.Tensor:
-        bs = self.block_size
-        return torch.tensor([block_ids[p // bs] * bs + p % bs for p in range(start, start + n)], dtype=torch.int32)
+        hf, _, _, _ = K.norm_fwd(hidden if rows is None else hidden[rows], e.w.p("final_norm"), eps=e.cfg.rms_eps)
+        return K.gemm(hf, e.w.p("lm_head"))
 
     # ------------------------------------------------------------------ prompt chunks
     @torch.no_grad()
-    def prefill_chunk(self, tokens: Sequence[int], start: int, block_ids: Sequence[int], want_token: bool) -> int:
+    def prefill_chunk(self, tokens: Sequence[int], start: int, block_ids: Sequence[int], want_token: bool, slot: int = 0) -> int:
         """Run prompt positions [start, start + len(tokens)) of one sequence: their K / V go into the sequence's blocks,
-        their queries attend to everything cached so far.  Returns the greedy next token when `want_token` (the chunk
-        completes the prompt), else -1."""
+        their queries attend to everything cached so far.  Returns the next token when `want_token` (the chunk completes
+        the prompt), else -1."""
         if self.prefix_cache_bytes > 0:
             return self._prefill_with_reuse(list(tokens), start, block_ids, want_token)
-        return self._prefill_compute(tokens, start, block_ids, want_token)
+        return super().prefill_chunk(tokens, start, block_ids, want_token)
 
     # ---- prefix reuse around the computation
     def _prefill_with_reuse(self, tokens: List[int], start: int, block_ids: Sequence[int], want_token: bool) -> int:
@@ -115,7 +102,7 @@ class LlamaKVModel:
                     self.cache.v[i][dst] = snap[1][i, b0:b1]
                 self.prefill_tokens_reused += m - start
                 covered = m
-        out = self._prefill_compute(sofar[covered:end], covered, block_ids, want_token) if covered < end else -1
+        out = super().prefill_chunk(sofar[covered:end], covered, block_ids, want_token) if covered < end else -1
         if want_token:
             self._seq_tokens.pop(key, None)
             self._remember(sofar, block_ids)
@@ -155,12 +142,10 @@ class LlamaKVModel:
         for n in sorted(lengths):                                 # the native index alone (it evicts by itself)
             self._index._lib.lt_prefix_insert(self._index._c, _i32(prompt[:n]), n, _i32([h]), 1)
 
-    @torch.no_grad()
-    def _prefill_compute(self, tokens: Sequence[int], start: int, block_ids: Sequence[int], want_token: bool) -> int:
+    def _prompt_hidden(self, tokens: Sequence[int], start: int, block_ids: Sequence[int], slot: int = 0):
         e, K = self.e, self.e.K
         dev = e.device
         n = len(tokens)
-        self.prefill_tokens_computed += n
         host = torch.empty(3, n, dtype=torch.int64)
         host[0] = torch.tensor(tokens, dtype=torch.int64)
         host[1] = torch.arange(start, start + n)
@@ -186,137 +171,21 @@ class LlamaKVModel:
             o, _ = K.flash_fwd(q.unsqueeze(0), kc.contiguous().unsqueeze(0), vc.contiguous().unsqueeze(0), causal=True)
             return o[0]
 
-        x = self._layers(K.embedding_fwd(tok, e.w.p("embed")), pos, attend)
-        if not want_token:
-            return -1
-        return int(self._next_tokens(x[-1:]).item())
+        return self._layers(K.embedding_fwd(tok, e.w.p("embed")), pos, attend)
 
     # ------------------------------------------------------------------ one token for every running sequence
-    def _decode_body(self, d: torch.Tensor, S: int, width: int) -> torch.Tensor:
-        """The device work of one decode step on the packed int64 input block `d` [4 + width, S]: rows 0-3 are token,
-        position, cache slot and context length of every sequence, the rest its block table (transposed)."""
+    def _decode_hidden(self, d: torch.Tensor, S: int, width: int) -> torch.Tensor:
         from ..serving import paged_attention
         e, K = self.e, self.e.K
         bs = self.block_size
         tok = d[0]
         pos, slots, ctx = d[1].to(torch.int32), d[2].to(torch.int32), d[3].to(torch.int32)
-        bt = d[4:].t().contiguous().to(torch.int32)
-        splits = self.num_splits or self._splits(S, width * bs)
+        bt = d[5:].t().contiguous().to(torch.int32)
+        splits = self.num_splits or self._splits_for(S * e.cfg.n_kv_heads, width * bs)
 
         def attend(i, q, k, v):
             self.cache.append(i, k.contiguous(), v.contiguous(), slots)
             return paged_attention(q.contiguous(), self.cache.k[i], self.cache.v[i], bt, ctx, bs, num_splits=splits,
                                    k_scale=self.cache.k_scale, v_scale=self.cache.v_scale)
 
-        x = self._layers(K.embedding_fwd(tok, e.w.p("embed")), pos, attend)
-        return self._next_tokens(x)
-
-    @torch.no_grad()
-    def decode_batch(self, last_tokens: Sequence[int], positions: Sequence[int], block_tables: List[Sequence[int]]) -> List[int]:
-        """last_tokens[s] sits at position positions[s] of sequence s and is not in the cache yet: append its K / V,
-        attend over positions[s] + 1 cached keys, return the greedy next token of every sequence.
-
-        On a GPU the step's ~270 launches are recorded once per (batch size, block-table width) into a CUDA graph and
-        replayed: the step then costs its kernels, not their launch overhead.  The inputs of a replay are copied
-        into the graph's static input block first."""
-        e = self.e
-        dev = e.device
-        S = len(last_tokens)
-        bs = self.block_size
-        width = max((p + bs) // bs for p in positions)
-        if self.graphs and dev.type == "cuda":
-            width = (width + 15) // 16 * 16                     # fewer distinct graphs: table widths in steps of 16 blocks
-        host = torch.zeros(4 + width, S, dtype=torch.int64)
-        host[0] = torch.tensor(list(last_tokens), dtype=torch.int64)
-        host[1] = torch.tensor(list(positions), dtype=torch.int64)
-        for s in range(S):
-            p = positions[s]
-            host[2, s] = block_tables[s][p // bs] * bs + p % bs
-            row = block_tables[s][:width]
-            host[4:4 + len(row), s] = torch.tensor(list(row), dtype=torch.int64)
-        host[3] = host[1] + 1
-        if not (self.graphs and dev.type == "cuda"):
-            return self._decode_body(host.to(dev, non_blocking=True), S, width).tolist()
-        key = (S, width)
-        entry = self._graphs.get(key)
-        if entry is None:
-            static_in = host.to(dev)
-            side = torch.cuda.Stream(device=dev)
-            side.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(side):                        # eager run on the capture stream: workspaces, caches
-                self._decode_body(static_in, S, width)
-            torch.cuda.current_stream().wait_stream(side)
-            torch.cuda.synchronize()
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g, stream=side):
-                static_out = self._decode_body(static_in, S, width)
-            entry = self._graphs[key] = (g, static_in, static_out)
-            # the two recording passes appended this step's K / V already; the replay below rewrites the same slots
-        g, static_in, static_out = entry
-        static_in.copy_(host, non_blocking=True)
-        g.replay()
-        return static_out.tolist()
-
-    def _splits(self, S: int, max_ctx: int) -> int:
-        """Splits of the key range per (sequence, KV head): about four CTAs per SM, at least 256 keys per split."""
-        ctas = S * self.e.cfg.n_kv_heads
-        return max(1, min(32, max_ctx // 256, (148 * 4 + ctas - 1) // ctas))
-
-
-class Sampler:
-    """Temperature / top-k / nucleus sampling of next tokens from logits [rows, vocab] with its own random generator, so
-    that a run is reproducible from its seed.  `temperature == 0` (or `top_k == 1`) is greedy."""
-
-    def __init__(self, temperature: float = 1.0, top_k: int = 0, top_p: float = 1.0, seed: int = 0, device="cpu"):
-        self.temperature, self.top_k, self.top_p = float(temperature), int(top_k), float(top_p)
-        self.gen = torch.Generator(device=device).manual_seed(int(seed))
-
-    def __call__(self, logits: torch.Tensor) -> torch.Tensor:
-        if self.temperature <= 0.0 or self.top_k == 1:
-            return logits.argmax(-1)
-        z = logits / self.temperature
-        if self.top_k > 0 and self.top_k < z.shape[-1]:
-            kth = z.topk(self.top_k, -1).values[..., -1:]
-            z = z.masked_fill(z < kth, float("-inf"))
-        if self.top_p < 1.0:
-            order = z.sort(-1, descending=True)
-            p = torch.softmax(order.values, -1)
-            before = p.cumsum(-1) - p                     # probability mass ahead of each token, in sorted order
-            drop = before >= self.top_p                   # the first token always stays
-            z = z.masked_fill(torch.zeros_like(drop).scatter(-1, order.indices, drop), float("-inf"))
-        return torch.multinomial(torch.softmax(z, -1), 1, generator=self.gen).squeeze(-1)
-
-
-@torch.no_grad()
-def generate(engine: LlamaEngine, prompts: Sequence[Sequence[int]], max_new_tokens: int, *, temperature: float = 0.0,
-             top_k: int = 0, top_p: float = 1.0, seed: int = 0, eos_id: int = -1, block_size: int = 16,
-             max_num_seqs: int = 64, max_num_batched_tokens: int = 4096, kv_dtype=None,
-             prefix_cache_bytes: int = 0) -> List[List[int]]:
-    """Continue every prompt by up to `max_new_tokens` tokens (stopping at `eos_id`) with continuous batching on a paged KV
-    cache sized for the request, and return the new tokens per prompt.  Greedy by default (the decode step is replayed
-    from CUDA graphs on a GPU); with `temperature > 0` the next tokens are drawn by `Sampler` (eager decode steps)."""
-    from ..serving import Request, ServingScheduler
-    cfg = engine.cfg
-    need = sum((len(p) + max_new_tokens + block_size - 1) // block_size for p in prompts)
-    greedy = temperature <= 0.0 or top_k == 1
-    if kv_dtype is None:
-        kv_dtype = torch.bfloat16 if engine.device.type == "cuda" else torch.float32
-    model = LlamaKVModel(engine, num_blocks=need + 1, block_size=block_size, kv_dtype=kv_dtype, graphs=greedy,
-                         prefix_cache_bytes=prefix_cache_bytes)   # prompts of one call that share a prefix reuse its blocks
-    if not greedy:
-        model.sampler = Sampler(temperature, top_k, top_p, seed, device=engine.device)
-    sched = ServingScheduler(num_blocks=need + 1, block_size=block_size, max_num_seqs=max_num_seqs,
-                             max_num_batched_tokens=max_num_batched_tokens, eos_id=eos_id)
-    reqs = [Request(i, list(p), max_new_tokens=max_new_tokens) for i, p in enumerate(prompts)]
-    for r in reqs:
-        if len(r.prompt_tokens) + max_new_tokens > cfg.max_seq:
-            raise ValueError("prompt %d: %d tokens + %d new exceed the model's %d positions" %
-                             (r.id, len(r.prompt_tokens), max_new_tokens, cfg.max_seq))
-        sched.add_request(r)
-    finished, guard = 0, 0
-    while finished < len(reqs):
-        finished += len(sched.step(model))
-        guard += 1
-        if guard > 4 * (max_new_tokens + len(reqs)) + 64 + sum(len(p) for p in prompts):
-            raise RuntimeError("the schedule did not finish")
-    return [list(r.generated_tokens) for r in reqs]
+        return self._layers(K.embedding_fwd(tok, e.w.p("embed")), pos, attend)

@@ -34,6 +34,9 @@ def _h():
         lib.lt_sched_tokens.argtypes = [c_void_p, c_int64, POINTER(c_int32), c_int, POINTER(c_int)]
         lib.lt_sched_block_table.argtypes = [c_void_p, c_int64, POINTER(c_int32), c_int]
         lib.lt_sched_context_len.argtypes = [c_void_p, c_int64]
+        for f in ("lt_sched_slot", "lt_sched_session_open", "lt_sched_session_close"):
+            getattr(lib, f).argtypes = [c_void_p, c_int64]
+        lib.lt_sched_session_grow.argtypes = [c_void_p, c_int64, c_int]
         lib.lt_sched_pop_finished.argtypes = [c_void_p, POINTER(c_int64), c_int]
         lib.lt_sched_release.argtypes = [c_void_p, c_int64]
         for f in ("lt_sched_num_free_blocks", "lt_sched_num_running", "lt_sched_num_pending"):
@@ -59,12 +62,27 @@ class PagedKVCache:
 
     def __init__(self, num_layers: int, num_blocks: int, block_size: int, n_kv_heads: int, head_dim: int, device="cuda",
                  dtype=torch.bfloat16, k_scale: float = 1.0, v_scale: float = 1.0):
-        self.block_size, self.n_kv_heads, self.head_dim = block_size, n_kv_heads, head_dim
+        self._init(num_blocks, block_size, [(n_kv_heads, head_dim, head_dim)] * num_layers, device, dtype, k_scale, v_scale)
+        self.n_kv_heads, self.head_dim = n_kv_heads, head_dim
+
+    @classmethod
+    def per_layer(cls, shapes, num_blocks: int, block_size: int, device="cuda", dtype=torch.bfloat16) -> "PagedKVCache":
+        """Layers that differ: `shapes` has (kv heads, key size, value size) of every layer, None for a layer that keeps no
+        keys.  All layers share the block tables."""
+        self = cls.__new__(cls)
+        self._init(num_blocks, block_size, shapes, device, dtype, 1.0, 1.0)
+        return self
+
+    def _init(self, num_blocks, block_size, shapes, device, dtype, k_scale, v_scale):
+        self.block_size = block_size
         self.fp8 = dtype == torch.float8_e4m3fn
         self.k_scale, self.v_scale = k_scale, v_scale
-        shape = (num_blocks, n_kv_heads, block_size, head_dim)
-        self.k = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
+        self.k = [None if s is None else torch.zeros((num_blocks, s[0], block_size, s[1]), dtype=dtype, device=device) for s in shapes]
+        self.v = [None if s is None else torch.zeros((num_blocks, s[0], block_size, s[2]), dtype=dtype, device=device) for s in shapes]
+
+    @property
+    def bytes_per_token(self) -> int:
+        return sum(t[0, :, 0].numel() * t.element_size() for t in self.k + self.v if t is not None)
 
     def append(self, layer: int, k_new: torch.Tensor, v_new: torch.Tensor, slots: torch.Tensor):
         """k_new / v_new: [N, Hkv, D]; slots: [N] int32 = block * block_size + offset."""
@@ -114,6 +132,32 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     return out.to(q.dtype)
 
 
+# ------------------------------------------------------------------------------------------------ recurrent state
+class RecurrentStatePool:
+    """fp32 state of recurrent layers, one row per active sequence: `pool[layer, name]` is [slots + 1, ...].  The scheduler
+    deals the slots out like cache blocks.  Nothing is cleared when a slot changes hands: kernels ignore what is there at
+    a sequence's first position.  The row after the last slot is scratch, for passes whose effect must not count."""
+
+    def __init__(self, slots: int, device="cuda"):
+        self.slots, self.device = slots, device
+        self._t: Dict[tuple, torch.Tensor] = {}
+
+    @property
+    def scratch(self) -> int:
+        return self.slots
+
+    def add(self, layer: int, name: str, *shape: int) -> torch.Tensor:
+        t = self._t[layer, name] = torch.zeros((self.slots + 1,) + shape, dtype=torch.float32, device=self.device)
+        return t
+
+    def __getitem__(self, key) -> torch.Tensor:
+        return self._t[key]
+
+    @property
+    def bytes_per_slot(self) -> int:
+        return sum(t[0].numel() * 4 for t in self._t.values())
+
+
 # ------------------------------------------------------------------------------------------------ scheduler
 class Request:
     def __init__(self, id: int, prompt: Sequence[int], max_new_tokens: int = 32):
@@ -124,6 +168,7 @@ class Request:
         self.prefill_processed = 0
         self.is_finished = False
         self.block_ids: List[int] = []
+        self.slot = -1                    # row of the per-sequence state while the request is active
 
 
 class _BlockCount(int):
@@ -143,6 +188,7 @@ class ServingScheduler:
         self._s = self._lib.lt_sched_create(num_blocks, block_size, max_num_seqs, max_num_batched_tokens, eos_id)
         self._reqs: Dict[int, Request] = {}
         self._order: List[int] = []
+        self._sessions: Dict[int, int] = {}          # session id -> tokens it has been given
 
     def __del__(self):
         try:
@@ -182,6 +228,7 @@ class ServingScheduler:
         bt = (c_int32 * 4096)()
         nb = self._lib.lt_sched_block_table(self._s, rid, bt, 4096)
         r.block_ids = [int(bt[i]) for i in range(min(nb, 4096))]
+        r.slot = self._lib.lt_sched_slot(self._s, rid)
         r.prefill_processed = min(self._lib.lt_sched_context_len(self._s, rid), len(r.prompt_tokens))
 
     def _tokens(self, rid: int) -> List[int]:
@@ -268,19 +315,21 @@ class ServingScheduler:
         if n == 0:
             return []
         dec = []
+        slots = getattr(model, "state_slots", 0) > 0          # recurrent layers: the sequence's state row goes along
         for i in range(n):
             rid, st, ln = int(ids[i]), int(starts[i]), int(lens[i])
             self._sync(rid)
             r = self._reqs[rid]
             if ln > 0:
                 done = st + ln >= len(r.prompt_tokens)
-                nxt = model.prefill_chunk(r.prompt_tokens[st:st + ln], st, r.block_ids, done)
+                nxt = model.prefill_chunk(r.prompt_tokens[st:st + ln], st, r.block_ids, done, **({"slot": r.slot} if slots else {}))
                 self._lib.lt_sched_commit(self._s, rid, int(nxt) if done else -1)
             else:
                 dec.append((rid, st))
         if dec:
             toks = [self._tokens(rid)[pos] for rid, pos in dec]
-            nxt = model.decode_batch(toks, [pos for _, pos in dec], [self._reqs[rid].block_ids for rid, _ in dec])
+            nxt = model.decode_batch(toks, [pos for _, pos in dec], [self._reqs[rid].block_ids for rid, _ in dec],
+                                     **({"slots": [self._reqs[rid].slot for rid, _ in dec]} if slots else {}))
             for (rid, _), t in zip(dec, nxt):
                 self._lib.lt_sched_commit(self._s, rid, int(t))
         fin = (c_int64 * cap)()
@@ -294,6 +343,46 @@ class ServingScheduler:
             out.append(r)
             self._retire(r.id)
         return out
+
+    # ---- sessions: the caller brings the tokens
+    def feed(self, model, entries) -> List[torch.Tensor]:
+        """One step over sequences whose tokens are given: entries are (session id, next tokens, rows); every session
+        continues from the cache and the state its earlier tokens left (a new id opens one).  Returns, per entry, the fp32
+        logits [len(rows), vocab] at those places among the entry's tokens.  Portions go through the model's prompt path,
+        single further tokens through one batched decode step; nothing is sampled."""
+        out: List[Optional[torch.Tensor]] = [None] * len(entries)
+        dec = []
+        kinds = []
+        for sid, tokens, rows in entries:                     # reserve first, so that a pool that is too small changes nothing
+            sid = int(sid)
+            if sid not in self._sessions:
+                if self._lib.lt_sched_session_open(self._s, sid) < 0:
+                    raise RuntimeError("no free state slot for session %d" % sid)
+                self._sessions[sid] = 0
+            start = self._sessions[sid]
+            nb = self._lib.lt_sched_session_grow(self._s, sid, start + len(tokens))
+            if nb < 0:
+                raise RuntimeError("the KV pool is too small for session %d at %d tokens" % (sid, start + len(tokens)))
+            bt = (c_int32 * max(nb, 1))()
+            self._lib.lt_sched_block_table(self._s, sid, bt, nb)
+            kinds.append((sid, start, [int(b) for b in bt[:nb]], self._lib.lt_sched_slot(self._s, sid)))
+        for i, ((_, tokens, rows), (sid, start, blocks, slot)) in enumerate(zip(entries, kinds)):
+            self._sessions[sid] = start + len(tokens)
+            if len(tokens) == 1 and start > 0:
+                dec.append(i)
+            elif len(tokens):
+                out[i] = model.score_chunk([int(t) for t in tokens], start, blocks, list(rows), slot=slot)
+        if dec:
+            logits = model.decode_logits([int(entries[i][1][0]) for i in dec], [kinds[i][1] for i in dec], [kinds[i][2] for i in dec],
+                                         slots=[kinds[i][3] for i in dec])
+            for row, i in enumerate(dec):
+                out[i] = logits[row:row + 1][:len(entries[i][2])]
+        return out
+
+    def end_session(self, sid: int) -> None:
+        """Blocks and slot of a session go back to the pools."""
+        if self._sessions.pop(int(sid), None) is not None:
+            self._lib.lt_sched_session_close(self._s, int(sid))
 
     def get_block_table_tensor(self) -> Tensor:
         run = self.running_queue
