@@ -57,6 +57,9 @@ def _parse():
     ap.add_argument("--hybrid", action="store_true",
                     help="with --tp 1: shard over dp with the FSDP x TP provider (weights prefetched by peer-pull kernels) "
                          "instead of the ZeRO-3 provider whose all-gather runs inside the GEMMs")
+    ap.add_argument("--serving-compare", action="store_true",
+                    help="instead of the training workload: prompt and decode throughput of Safuvik models beside Llama models of equal "
+                         "size, and their kernels (litetorch_b200.utils.hybrid_bench; prints JSON lines and tables)")
     return ap.parse_args()
 
 
@@ -420,7 +423,10 @@ def run_reference(args):
 
 if __name__ == "__main__":
     a = _parse()
-    if a.impl == "reference":
+    if a.serving_compare:
+        from litetorch_b200.utils import hybrid_bench
+        hybrid_bench.main([])
+    elif a.impl == "reference":
         run_reference(a)
     else:
         run_ours(a)

@@ -57,53 +57,58 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, TO* __restric
     }
 }
 
-// y[R, J] (fp32) = x[R, K] @ w[J, K]^T for a narrow w: a CTA takes four rows, its eight warps share the J columns, two at
-// a time, so that a row of w is read once per four rows of x.
-constexpr int kRdRows = 4;
+// y[R, J] (fp32) = x[R, K] @ w[J, K]^T for a narrow w: a CTA makes a 4 x 4 patch, its eight warps share K (so that a
+// handful of rows is not bound by the latency of one long walk) and fold their sums through shared memory.
+constexpr int kRdTile = 4;
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
 rows_dot_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, float* __restrict__ y, int R, int J, int K) {
+  __shared__ float part[8][kRdTile * kRdTile];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int r0 = blockIdx.x * kRdRows;
-  for (int j = (blockIdx.y * 8 + warp) * 2; j < J; j += gridDim.y * 16) {
-    const bool two = j + 1 < J;
-    float acc[2][kRdRows] = {};
-    for (int k = lane * V; k < K; k += 32 * V) {
-      float wv[2][V];
+  const int r0 = blockIdx.x * kRdTile, j0 = blockIdx.y * kRdTile;
+  const T* xp[kRdTile];
+  const T* wp[kRdTile];
+#pragma unroll
+  for (int i = 0; i < kRdTile; ++i) {            // rows past the end read the last row; their results are dropped
+    xp[i] = x + min(r0 + i, R - 1) * ldx;
+    wp[i] = w + (long long)min(j0 + i, J - 1) * K;
+  }
+  float acc[kRdTile][kRdTile] = {};
+#pragma unroll 2
+  for (int k = threadIdx.x * V; k < K; k += 256 * V) {
+    float xv[kRdTile][V], wv[kRdTile][V];
+#pragma unroll
+    for (int i = 0; i < kRdTile; ++i) {
       if constexpr (V == 4) {
-        const float4 a = ldf4(w + (long long)j * K + k);
-        const float4 b = two ? ldf4(w + (long long)(j + 1) * K + k) : make_float4(0.f, 0.f, 0.f, 0.f);
-        wv[0][0] = a.x; wv[0][1] = a.y; wv[0][2] = a.z; wv[0][3] = a.w;
-        wv[1][0] = b.x; wv[1][1] = b.y; wv[1][2] = b.z; wv[1][3] = b.w;
+        const float4 a = ldf4(xp[i] + k), b = ldf4(wp[i] + k);
+        xv[i][0] = a.x; xv[i][1] = a.y; xv[i][2] = a.z; xv[i][3] = a.w;
+        wv[i][0] = b.x; wv[i][1] = b.y; wv[i][2] = b.z; wv[i][3] = b.w;
       } else {
-        wv[0][0] = ldf(w + (long long)j * K + k);
-        wv[1][0] = two ? ldf(w + (long long)(j + 1) * K + k) : 0.f;
-      }
-#pragma unroll
-      for (int r = 0; r < kRdRows; ++r) {
-        if (r0 + r >= R) break;
-        float xv[V];
-        if constexpr (V == 4) {
-          const float4 a = ldf4(x + (r0 + r) * ldx + k);
-          xv[0] = a.x; xv[1] = a.y; xv[2] = a.z; xv[3] = a.w;
-        } else {
-          xv[0] = ldf(x + (r0 + r) * ldx + k);
-        }
-#pragma unroll
-        for (int v = 0; v < V; ++v) {
-          acc[0][r] = fmaf(wv[0][v], xv[v], acc[0][r]);
-          acc[1][r] = fmaf(wv[1][v], xv[v], acc[1][r]);
-        }
+        xv[i][0] = ldf(xp[i] + k);
+        wv[i][0] = ldf(wp[i] + k);
       }
     }
 #pragma unroll
-    for (int r = 0; r < kRdRows; ++r) {
-      const float a = warp_sum(acc[0][r]), b = warp_sum(acc[1][r]);
-      if (lane == 0 && r0 + r < R) {
-        y[(long long)(r0 + r) * J + j] = a;
-        if (two) y[(long long)(r0 + r) * J + j + 1] = b;
-      }
+    for (int r = 0; r < kRdTile; ++r)
+#pragma unroll
+      for (int c = 0; c < kRdTile; ++c)
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[r][c] = fmaf(xv[r][v], wv[c][v], acc[r][c]);
+  }
+#pragma unroll
+  for (int r = 0; r < kRdTile; ++r)
+#pragma unroll
+    for (int c = 0; c < kRdTile; ++c) {
+      const float v = warp_sum(acc[r][c]);
+      if (lane == 0) part[warp][r * kRdTile + c] = v;
     }
+  __syncthreads();
+  if (threadIdx.x < kRdTile * kRdTile) {
+    const int r = r0 + threadIdx.x / kRdTile, c = j0 + threadIdx.x % kRdTile;
+    float v = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v += part[i][threadIdx.x];
+    if (r < R && c < J) y[(long long)r * J + c] = v;
   }
 }
 
@@ -135,10 +140,8 @@ int lt_gemm_simt(int in_fp32, int out_fp32, const void* A, const void* B, void* 
 int lt_rows_dot(int fp32, const void* x, long long ldx, const void* w, float* y, int R, int J, int K, void* stream) {
   using namespace lt;
   if (R <= 0 || J <= 0) return 0;
-  const int rb = (R + kRdRows - 1) / kRdRows;
-  int jb = 1;
-  if (rb < 148) jb = (J + 15) / 16;
-  dim3 grid(rb, jb);
+  dim3 grid((R + kRdTile - 1) / kRdTile, (J + kRdTile - 1) / kRdTile);
+  if (grid.y > 65535) return -4;
   const bool v4 = K % 4 == 0 && ldx % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   using bf = __nv_bfloat16;

@@ -38,6 +38,7 @@ __global__ void __launch_bounds__(256)
 mlstm_gates_kernel(const float* __restrict__ logits, const float* __restrict__ ib, const float* __restrict__ fb, float cap,
                    const float* __restrict__ m_state, float* __restrict__ a_out, float* __restrict__ f_out,
                    float* __restrict__ c_out, float* __restrict__ m_out, int N, int H, int chunks) {
+  extern __shared__ float last_s[];      // [chunks] F at a chunk's last token, [chunks] largest a of the chunk
   const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float bi = ib[h], bf = fb[h];
   for (int c = warp; c < chunks; c += 8) {
@@ -72,14 +73,15 @@ mlstm_gates_kernel(const float* __restrict__ logits, const float* __restrict__ i
       run = __shfl_sync(0xffffffffu, f, 31);
       top = __shfl_sync(0xffffffffu, mx, 31);
     }
+    // (tokens past the end add nothing to F and -inf to the maximum)
+    if (lane == 0) { last_s[c] = run; last_s[chunks + c] = top; }
   }
   __syncthreads();
   if (threadIdx.x == 0) {
     float m = m_state ? m_state[h] : 0.f;
     for (int c = 0; c < chunks; ++c) {
       m_out[(long long)h * (chunks + 1) + c] = m;
-      const int last = min(N, (c + 1) * kMlChunk) - 1;
-      m = f_out[(long long)h * N + last] + fmaxf(m, c_out[(long long)h * N + last]);
+      m = last_s[c] + fmaxf(m, last_s[chunks + c]);
     }
     m_out[(long long)h * (chunks + 1) + chunks] = m;
   }
@@ -124,36 +126,39 @@ __device__ __forceinline__ uint4 load8(const __nv_bfloat16* row, int c, int cols
   return v;
 }
 
-// rows x 64 tile of a [.., ld] bf16 matrix into shared memory.
-__device__ __forceinline__ void load_tile(__nv_bfloat16* dst, const __nv_bfloat16* src, long long ld, int rows, int rows_ok, int c0,
-                                          int cols, bool aligned) {
-  for (int i = threadIdx.x; i < rows * 8; i += blockDim.x) {
-    const int r = i >> 3, c = (i & 7) * 8;
-    *reinterpret_cast<uint4*>(dst + r * kMlPitch + c) = load8(src + r * ld, c0 + c, cols, r < rows_ok, aligned);
-  }
-}
-
 // ------------------------------------------------------------------------------------------------ chunk states
-// U[h, c] [D, E] = sum_s exp(a_s - M_last) k_s v_s^T and nU[h, c] [D]; one CTA per 64 x 64 tile.
-__global__ void __launch_bounds__(128)
+// U[h, c] [D, E] = sum_s exp(a_s - M_last) k_s v_s^T and nU[h, c] [D].  One CTA per 64 rows of U: the decayed keys are split
+// into their two parts once and stay in shared memory while 128 columns of V at a time pass by (the next ones are loaded
+// into registers under the products).  Eight warps as 2 row halves x 4 column quarters of 32 x 32.
+constexpr int kMlWide = 128, kMlWidePitch = kMlWide + 8;
+constexpr size_t kMlStateSmem = (2 * size_t(kMlChunk) * kMlPitch + size_t(kMlChunk) * kMlWidePitch) * 2;
+
+__global__ void __launch_bounds__(256, 2)
 mlstm_chunk_state_kernel(const __nv_bfloat16* __restrict__ k, const __nv_bfloat16* __restrict__ v, long long ld,
                          const float* __restrict__ a, const float* __restrict__ cmax, const float* __restrict__ m_start,
                          float* __restrict__ U, float* __restrict__ nU, int N, int D, int E, int chunks, int aligned) {
   extern __shared__ __align__(16) uint8_t ml_smem[];
   __nv_bfloat16* kh = reinterpret_cast<__nv_bfloat16*>(ml_smem);          // [128][pitch]: high parts of w_s k_s
   __nv_bfloat16* kl = kh + kMlChunk * kMlPitch;
-  __nv_bfloat16* vs = kl + kMlChunk * kMlPitch;
+  __nv_bfloat16* vs = kl + kMlChunk * kMlPitch;                            // [128][wide pitch]
   __shared__ float w_s[kMlChunk];
-  const int c = blockIdx.x, h = blockIdx.y;
-  const int et = (E + kMlRows - 1) / kMlRows;
-  const int d0 = int(blockIdx.z / et) * kMlRows, e0 = int(blockIdx.z % et) * kMlRows;
+  const int c = blockIdx.x, h = blockIdx.y, d0 = blockIdx.z * kMlRows;
   const int t0 = c * kMlChunk, len = min(kMlChunk, N - t0);
   const float m_last = fmaxf(m_start[(long long)h * (chunks + 1) + c], cmax[(long long)h * N + t0 + len - 1]);
   if (int(threadIdx.x) < kMlChunk) w_s[threadIdx.x] = int(threadIdx.x) < len ? expf(a[(long long)h * N + t0 + threadIdx.x] - m_last) : 0.f;
-  __syncthreads();
   const __nv_bfloat16* kp = k + (long long)t0 * ld + (long long)h * D;
   const __nv_bfloat16* vp = v + (long long)t0 * ld + (long long)h * E;
-  for (int i = threadIdx.x; i < kMlChunk * 8; i += blockDim.x) {
+  uint4 vr[8];
+  auto fetch = [&](int e0) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int i = threadIdx.x + j * 256, r = i >> 4, cc = (i & 15) * 8;
+      vr[j] = load8(vp + r * ld, e0 + cc, E, r < len, aligned);
+    }
+  };
+  fetch(0);
+  __syncthreads();
+  for (int i = threadIdx.x; i < kMlChunk * 8; i += 256) {
     const int r = i >> 3, cc = (i & 7) * 8;
     const uint4 raw = load8(kp + r * ld, d0 + cc, D, r < len, aligned);
     const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&raw);
@@ -164,41 +169,58 @@ mlstm_chunk_state_kernel(const __nv_bfloat16* __restrict__ k, const __nv_bfloat1
     *reinterpret_cast<uint4*>(kh + r * kMlPitch + cc) = hi;
     *reinterpret_cast<uint4*>(kl + r * kMlPitch + cc) = lo;
   }
-  load_tile(vs, vp, ld, kMlChunk, len, e0, E, aligned);
-  __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lj = lane >> 3, lr = lane & 7;
-  const int wd = (warp >> 1) * 32, we = (warp & 1) * 32;
-  float acc[2][4][4] = {};
+  const int wd = (warp >> 2) * 32, we = (warp & 3) * 32;
+  const int g = lane >> 2, q = lane & 3;
+  float* out = U + ((long long)h * chunks + c) * D * E;
+  const bool e2 = (E & 1) == 0;
+  for (int e0 = 0; e0 < E; e0 += kMlWide) {
 #pragma unroll
-  for (int ks = 0; ks < kMlChunk; ks += 16) {
-    uint32_t b[2][4];
+    for (int j = 0; j < 8; ++j) {
+      const int i = threadIdx.x + j * 256, r = i >> 4, cc = (i & 15) * 8;
+      *reinterpret_cast<uint4*>(vs + r * kMlWidePitch + cc) = vr[j];
+    }
+    __syncthreads();
+    if (e0 + kMlWide < E) fetch(e0 + kMlWide);
+    float acc[2][4][4] = {};
 #pragma unroll
-    for (int nb = 0; nb < 2; ++nb) ldsm4t(vs + (ks + (lj & 1) * 8 + lr) * kMlPitch + we + nb * 16 + (lj >> 1) * 8, b[nb]);
+    for (int ks = 0; ks < kMlChunk; ks += 16) {
+      uint32_t b[2][4];
 #pragma unroll
-    for (int mb = 0; mb < 2; ++mb) {
-      const int off = (ks + (lj >> 1) * 8 + lr) * kMlPitch + wd + mb * 16 + (lj & 1) * 8;
-      uint32_t ah[4], al[4];
-      ldsm4t(kh + off, ah);
-      ldsm4t(kl + off, al);
+      for (int nb = 0; nb < 2; ++nb) ldsm4t(vs + (ks + (lj & 1) * 8 + lr) * kMlWidePitch + we + nb * 16 + (lj >> 1) * 8, b[nb]);
 #pragma unroll
-      for (int nb = 0; nb < 4; ++nb) {
-        mma16816(acc[mb][nb], ah, b[nb >> 1][(nb & 1) * 2], b[nb >> 1][(nb & 1) * 2 + 1]);
-        mma16816(acc[mb][nb], al, b[nb >> 1][(nb & 1) * 2], b[nb >> 1][(nb & 1) * 2 + 1]);
+      for (int mb = 0; mb < 2; ++mb) {
+        const int off = (ks + (lj >> 1) * 8 + lr) * kMlPitch + wd + mb * 16 + (lj & 1) * 8;
+        uint32_t ah[4], al[4];
+        ldsm4t(kh + off, ah);
+        ldsm4t(kl + off, al);
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) {
+          mma16816(acc[mb][nb], ah, b[nb >> 1][(nb & 1) * 2], b[nb >> 1][(nb & 1) * 2 + 1]);
+          mma16816(acc[mb][nb], al, b[nb >> 1][(nb & 1) * 2], b[nb >> 1][(nb & 1) * 2 + 1]);
+        }
       }
     }
+#pragma unroll
+    for (int mb = 0; mb < 2; ++mb)
+#pragma unroll
+      for (int nb = 0; nb < 4; ++nb)
+#pragma unroll
+        for (int r = 0; r < 4; r += 2) {
+          const int d = d0 + wd + mb * 16 + g + (r >> 1) * 8, e = e0 + we + nb * 8 + q * 2;
+          if (d < D && e < E) {
+            float* dst = out + (long long)d * E + e;
+            if (e2) {
+              *reinterpret_cast<float2*>(dst) = make_float2(acc[mb][nb][r], acc[mb][nb][r + 1]);
+            } else {
+              dst[0] = acc[mb][nb][r];
+              if (e + 1 < E) dst[1] = acc[mb][nb][r + 1];
+            }
+          }
+        }
+    __syncthreads();
   }
-  float* out = U + ((long long)h * chunks + c) * D * E;
-  const int g = lane >> 2, q = lane & 3;
-#pragma unroll
-  for (int mb = 0; mb < 2; ++mb)
-#pragma unroll
-    for (int nb = 0; nb < 4; ++nb)
-#pragma unroll
-      for (int r = 0; r < 4; ++r) {
-        const int d = d0 + wd + mb * 16 + g + (r >> 1) * 8, e = e0 + we + nb * 8 + q * 2 + (r & 1);
-        if (d < D && e < E) out[(long long)d * E + e] = acc[mb][nb][r];
-      }
-  if (e0 == 0 && threadIdx.x < kMlRows && d0 + int(threadIdx.x) < D) {
+  if (threadIdx.x < kMlRows && d0 + int(threadIdx.x) < D) {
     float s = 0.f;
     for (int r = 0; r < len; ++r)
       s += __bfloat162float(kh[r * kMlPitch + threadIdx.x]) + __bfloat162float(kl[r * kMlPitch + threadIdx.x]);
@@ -208,7 +230,6 @@ mlstm_chunk_state_kernel(const __nv_bfloat16* __restrict__ k, const __nv_bfloat1
 
 // ------------------------------------------------------------------------------------------------ scan over chunks
 // In place: U[h, c] becomes the state at the start of chunk c; the state after the last chunk goes back to the slot.
-// Element index runs over D * E values of S and then D of n.
 template <int V>
 __global__ void __launch_bounds__(256)
 mlstm_chunk_scan_kernel(float* __restrict__ U, float* __restrict__ nU, const float* __restrict__ cmax,
@@ -224,48 +245,49 @@ mlstm_chunk_scan_kernel(float* __restrict__ U, float* __restrict__ nU, const flo
   if (blockIdx.x == 0 && threadIdx.x == 0) m_out[h] = m_start[(long long)h * (chunks + 1) + chunks];
   __syncthreads();
   const long long DE = (long long)D * E;
-  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
-  if (i < DE) {
-    float* u = U + (long long)h * chunks * DE + i;
-    float* st = S + (long long)h * DE + i;
-    if constexpr (V == 4) {
-      float4 cur = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
-      float4 nx[4];
-      for (int c0 = 0; c0 < chunks; c0 += 4) {
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (c0 + j < chunks) nx[j] = *reinterpret_cast<const float4*>(u + (c0 + j) * DE);
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (c0 + j < chunks) {
-            *reinterpret_cast<float4*>(u + (c0 + j) * DE) = cur;
-            const float k = keep_s[c0 + j];
-            cur = make_float4(fmaf(k, cur.x, nx[j].x), fmaf(k, cur.y, nx[j].y), fmaf(k, cur.z, nx[j].z), fmaf(k, cur.w, nx[j].w));
-          }
+  const unsigned s_blocks = unsigned((DE + 256 * V - 1) / (256 * V));        // the blocks after these take n
+  // One column of V values through all chunks: eight chunks are read ahead of their use.
+  auto walk = [&](float* u, long long stride, const float* first, float* last) {
+    float cur[V], nx[8][V];
+    auto ld = [&](const float* p, float (&d)[V]) {
+      if constexpr (V == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(p);
+        d[0] = f.x; d[1] = f.y; d[2] = f.z; d[3] = f.w;
+      } else {
+        d[0] = *p;
       }
-      *reinterpret_cast<float4*>(st) = cur;
+    };
+    auto st = [&](float* p, const float (&d)[V]) {
+      if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(d[0], d[1], d[2], d[3]);
+      else *p = d[0];
+    };
+    if (fresh) {
+#pragma unroll
+      for (int v = 0; v < V; ++v) cur[v] = 0.f;
     } else {
-      float cur = fresh ? 0.f : *st;
-      for (int c = 0; c < chunks; ++c) {
-        const float x = u[c * DE];
-        u[c * DE] = cur;
-        cur = fmaf(keep_s[c], cur, x);
-      }
-      *st = cur;
+      ld(first, cur);
     }
+    for (int c0 = 0; c0 < chunks; c0 += 8) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (c0 + j < chunks) ld(u + (c0 + j) * stride, nx[j]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (c0 + j < chunks) {
+          st(u + (c0 + j) * stride, cur);
+          const float k = keep_s[c0 + j];
+#pragma unroll
+          for (int v = 0; v < V; ++v) cur[v] = fmaf(k, cur[v], nx[j][v]);
+        }
+    }
+    st(last, cur);
+  };
+  if (blockIdx.x < s_blocks) {
+    const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * V;
+    if (i < DE) walk(U + (long long)h * chunks * DE + i, DE, S + (long long)h * DE + i, S + (long long)h * DE + i);
   } else {
-    for (int v = 0; v < V; ++v) {
-      const long long d = i - DE + v;
-      if (d >= D) break;
-      float cur = fresh ? 0.f : n_in[(long long)h * D + d];
-      float* u = nU + (long long)h * chunks * D + d;
-      for (int c = 0; c < chunks; ++c) {
-        const float x = u[(long long)c * D];
-        u[(long long)c * D] = cur;
-        cur = fmaf(keep_s[c], cur, x);
-      }
-      n_out[(long long)h * D + d] = cur;
-    }
+    const long long d = ((long long)(blockIdx.x - s_blocks) * 256 + threadIdx.x) * V;
+    if (d < D) walk(nU + (long long)h * chunks * D + d, D, n_in + (long long)h * D + d, n_out + (long long)h * D + d);
   }
 }
 
@@ -293,7 +315,7 @@ struct MlstmOut {
 constexpr int kMlPPitch = kMlChunk + 8;
 static size_t mlstm_out_smem(int D) {
   const int dp = (D + 63) / 64 * 64 + 8;
-  return size_t(kMlRows) * dp * 2 + 2 * size_t(kMlRows) * kMlPPitch * 2 + 2 * size_t(kMlRows) * kMlPitch * 2;
+  return size_t(kMlRows) * dp * 2 + 2 * size_t(kMlRows) * kMlPPitch * 2 + 4 * size_t(kMlRows) * kMlPitch * 2;
 }
 
 // One CTA: 64 tokens (half a chunk) of one head, eight warps as 4 row blocks of 16 x 2 column halves of 32.
@@ -304,8 +326,7 @@ __global__ void __launch_bounds__(256, 2) mlstm_out_kernel(const MlstmOut p) {
   __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(ml_smem);      // [64][dp]
   __nv_bfloat16* ph = qs + kMlRows * dp;                               // [64][kMlPPitch] token weights, high and low parts
   __nv_bfloat16* pl = ph + kMlRows * kMlPPitch;
-  __nv_bfloat16* t0s = pl + kMlRows * kMlPPitch;                       // two 64 x 64 tiles
-  __nv_bfloat16* t1s = t0s + kMlRows * kMlPitch;
+  __nv_bfloat16* tiles = pl + kMlRows * kMlPPitch;                     // two buffers of two 64 x 64 tiles (high and low parts)
   __shared__ float a_s[kMlChunk], top_s[kMlRows], inter_s[kMlRows], den_s[2][kMlRows], inv_s[kMlRows], sq_s[2][kMlRows];
   const int h = blockIdx.y, c = blockIdx.x >> 1, half = blockIdx.x & 1;
   const int t0 = c * kMlChunk, r0 = half * kMlRows;                    // chunk start, first row inside it
@@ -331,23 +352,52 @@ __global__ void __launch_bounds__(256, 2) mlstm_out_kernel(const MlstmOut p) {
   }
   __syncthreads();
 
+  // Tiles come through registers: the next one is loaded while the current one is multiplied, then stored into the other
+  // buffer, so that a tile costs one barrier.
+  constexpr int kTile = kMlRows * kMlPitch;
+  uint4 reg[4];
+  auto fetch_bf = [&](const __nv_bfloat16* src, int rows_ok, int c0, int cols) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = threadIdx.x + j * 256, r = i >> 3;
+      reg[j] = load8(src + r * p.ld, c0 + (i & 7) * 8, cols, r < rows_ok, p.aligned);
+    }
+  };
+  auto store_bf = [&](__nv_bfloat16* dst) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = threadIdx.x + j * 256;
+      *reinterpret_cast<uint4*>(dst + (i >> 3) * kMlPitch + (i & 7) * 8) = reg[j];
+    }
+  };
+  const int nd = (D + 63) / 64;
+
   // ---- token weights: (q . k) qscale exp(a_s - M_t) for s <= t, and their row sums
   float sum_lo = 0.f, sum_hi = 0.f;
-  for (int kb = 0; kb <= half; ++kb) {
+  const __nv_bfloat16* kp = p.k + (long long)t0 * p.ld + (long long)h * D;
+  const int k_stages = (half + 1) * nd;
+  auto fetch_k = [&](int st) {
+    const int kb = st / nd;
+    fetch_bf(kp + (long long)kb * kMlRows * p.ld, len - kb * kMlRows, (st % nd) * 64, D);
+  };
+  fetch_k(0);
+  store_bf(tiles);
+  __syncthreads();
+  for (int kb = 0, st = 0; kb <= half; ++kb) {
     float acc[4][4] = {};
-    const __nv_bfloat16* kp = p.k + (long long)(t0 + kb * kMlRows) * p.ld + (long long)h * D;
-    for (int d0 = 0; d0 < D; d0 += 64) {
-      load_tile(t0s, kp, p.ld, kMlRows, len - kb * kMlRows, d0, D, p.aligned);
-      __syncthreads();
+    for (int dd = 0; dd < nd; ++dd, ++st) {
+      if (st + 1 < k_stages) fetch_k(st + 1);
+      const __nv_bfloat16* t = tiles + (st & 1) * 2 * kTile;
 #pragma unroll
       for (int ks = 0; ks < 64; ks += 16) {
         uint32_t a[4], b[2][4];
-        ldsm4(qs + (wr + (lj & 1) * 8 + lr) * dp + d0 + ks + (lj >> 1) * 8, a);
+        ldsm4(qs + (wr + (lj & 1) * 8 + lr) * dp + dd * 64 + ks + (lj >> 1) * 8, a);
 #pragma unroll
-        for (int nb = 0; nb < 2; ++nb) ldsm4(t0s + (wc + nb * 16 + (lj >> 1) * 8 + lr) * kMlPitch + ks + (lj & 1) * 8, b[nb]);
+        for (int nb = 0; nb < 2; ++nb) ldsm4(t + (wc + nb * 16 + (lj >> 1) * 8 + lr) * kMlPitch + ks + (lj & 1) * 8, b[nb]);
 #pragma unroll
         for (int nb = 0; nb < 4; ++nb) mma16816(acc[nb], a, b[nb >> 1][(nb & 1) * 2], b[nb >> 1][(nb & 1) * 2 + 1]);
       }
+      if (st + 1 < k_stages) store_bf(tiles + ((st + 1) & 1) * 2 * kTile);
       __syncthreads();
     }
 #pragma unroll
@@ -384,76 +434,102 @@ __global__ void __launch_bounds__(256, 2) mlstm_out_kernel(const MlstmOut p) {
   }
   __syncthreads();
 
-  // ---- outputs, 64 columns at a time
+  // ---- outputs, 64 columns at a time: the state before the chunk (nd slices of it), then the chunk's own tokens
   float sq_lo = 0.f, sq_hi = 0.f;
   const float* S0 = p.S0 + ((long long)h * p.chunks + c) * D * E;
+  const __nv_bfloat16* vp = p.v + (long long)t0 * p.ld + (long long)h * E;
   const bool e4 = E % 4 == 0;
-  for (int e0 = 0; e0 < E; e0 += kMlRows) {
-    float acc[4][4] = {};
-    if (have_state) {
-      for (int d0 = 0; d0 < D; d0 += 64) {
-        for (int i = threadIdx.x; i < 64 * 16; i += 256) {
-          const int r = i >> 4, cc = (i & 15) * 4;
-          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (d0 + r < D && e0 + cc < E) {
-            const float* src = S0 + (long long)(d0 + r) * E + e0 + cc;
-            if (e4) {
-              v = *reinterpret_cast<const float4*>(src);
-            } else {
-              v.x = src[0];
-              if (e0 + cc + 1 < E) v.y = src[1];
-              if (e0 + cc + 2 < E) v.z = src[2];
-              if (e0 + cc + 3 < E) v.w = src[3];
-            }
-          }
-          split4(v, t0s + r * kMlPitch + cc, t1s + r * kMlPitch + cc);
+  const int ns = have_state ? nd : 0, per = ns + half + 1;
+  const int o_stages = ((E + 63) / 64) * per;
+  auto fetch_o = [&](int st) {
+    const int e0 = (st / per) * 64, k = st % per;
+    if (k >= ns) {
+      fetch_bf(vp + (long long)(k - ns) * kMlRows * p.ld, len - (k - ns) * kMlRows, e0, E);
+      return;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = threadIdx.x + j * 256, r = k * 64 + (i >> 4), cc = e0 + (i & 15) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < D && cc < E) {
+        const float* src = S0 + (long long)r * E + cc;
+        if (e4) {
+          v = *reinterpret_cast<const float4*>(src);
+        } else {
+          v.x = src[0];
+          if (cc + 1 < E) v.y = src[1];
+          if (cc + 2 < E) v.z = src[2];
+          if (cc + 3 < E) v.w = src[3];
         }
-        __syncthreads();
+      }
+      reg[j] = make_uint4(__float_as_uint(v.x), __float_as_uint(v.y), __float_as_uint(v.z), __float_as_uint(v.w));
+    }
+  };
+  auto store_o = [&](int st) {
+    __nv_bfloat16* t = tiles + (st & 1) * 2 * kTile;
+    if (st % per >= ns) {
+      store_bf(t);
+      return;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = threadIdx.x + j * 256, off = (i >> 4) * kMlPitch + (i & 15) * 4;
+      split4(make_float4(__uint_as_float(reg[j].x), __uint_as_float(reg[j].y), __uint_as_float(reg[j].z), __uint_as_float(reg[j].w)), t + off,
+             t + kTile + off);
+    }
+  };
+  fetch_o(0);
+  store_o(0);
+  __syncthreads();
+  for (int e0 = 0, st = 0; e0 < E; e0 += 64) {
+    float acc[4][4] = {};
+    for (int k = 0; k < per; ++k, ++st) {
+      if (st + 1 < o_stages) fetch_o(st + 1);
+      const __nv_bfloat16* t = tiles + (st & 1) * 2 * kTile;
+      if (k < ns) {
 #pragma unroll
         for (int ks = 0; ks < 64; ks += 16) {
           uint32_t a[4];
-          ldsm4(qs + (wr + (lj & 1) * 8 + lr) * dp + d0 + ks + (lj >> 1) * 8, a);
+          ldsm4(qs + (wr + (lj & 1) * 8 + lr) * dp + k * 64 + ks + (lj >> 1) * 8, a);
 #pragma unroll
           for (int nb = 0; nb < 2; ++nb) {
             uint32_t bh[4], bl[4];
             const int off = (ks + (lj & 1) * 8 + lr) * kMlPitch + wc + nb * 16 + (lj >> 1) * 8;
-            ldsm4t(t0s + off, bh);
-            ldsm4t(t1s + off, bl);
+            ldsm4t(t + off, bh);
+            ldsm4t(t + kTile + off, bl);
             mma16816(acc[nb * 2], a, bh[0], bh[1]);
             mma16816(acc[nb * 2 + 1], a, bh[2], bh[3]);
             mma16816(acc[nb * 2], a, bl[0], bl[1]);
             mma16816(acc[nb * 2 + 1], a, bl[2], bl[3]);
           }
         }
-        __syncthreads();
-      }
-      const float il = inter_s[wr + g], ih = inter_s[wr + g + 8];
+        if (k == ns - 1) {
+          const float il = inter_s[wr + g], ih = inter_s[wr + g + 8];
 #pragma unroll
-      for (int nb = 0; nb < 4; ++nb) {
-        acc[nb][0] *= il; acc[nb][1] *= il;
-        acc[nb][2] *= ih; acc[nb][3] *= ih;
-      }
-    }
-    const __nv_bfloat16* vp = p.v + (long long)t0 * p.ld + (long long)h * E;
-    for (int kb = 0; kb <= half; ++kb) {
-      load_tile(t0s, vp + (long long)kb * kMlRows * p.ld, p.ld, kMlRows, len - kb * kMlRows, e0, E, p.aligned);
-      __syncthreads();
+          for (int nb = 0; nb < 4; ++nb) {
+            acc[nb][0] *= il; acc[nb][1] *= il;
+            acc[nb][2] *= ih; acc[nb][3] *= ih;
+          }
+        }
+      } else {
 #pragma unroll
-      for (int ks = 0; ks < 64; ks += 16) {
-        uint32_t ah[4], al[4];
-        const int aoff = (wr + (lj & 1) * 8 + lr) * kMlPPitch + kb * kMlRows + ks + (lj >> 1) * 8;
-        ldsm4(ph + aoff, ah);
-        ldsm4(pl + aoff, al);
+        for (int ks = 0; ks < 64; ks += 16) {
+          uint32_t ah[4], al[4];
+          const int aoff = (wr + (lj & 1) * 8 + lr) * kMlPPitch + (k - ns) * kMlRows + ks + (lj >> 1) * 8;
+          ldsm4(ph + aoff, ah);
+          ldsm4(pl + aoff, al);
 #pragma unroll
-        for (int nb = 0; nb < 2; ++nb) {
-          uint32_t b[4];
-          ldsm4t(t0s + (ks + (lj & 1) * 8 + lr) * kMlPitch + wc + nb * 16 + (lj >> 1) * 8, b);
-          mma16816(acc[nb * 2], ah, b[0], b[1]);
-          mma16816(acc[nb * 2 + 1], ah, b[2], b[3]);
-          mma16816(acc[nb * 2], al, b[0], b[1]);
-          mma16816(acc[nb * 2 + 1], al, b[2], b[3]);
+          for (int nb = 0; nb < 2; ++nb) {
+            uint32_t b[4];
+            ldsm4t(t + (ks + (lj & 1) * 8 + lr) * kMlPitch + wc + nb * 16 + (lj >> 1) * 8, b);
+            mma16816(acc[nb * 2], ah, b[0], b[1]);
+            mma16816(acc[nb * 2 + 1], ah, b[2], b[3]);
+            mma16816(acc[nb * 2], al, b[0], b[1]);
+            mma16816(acc[nb * 2 + 1], al, b[2], b[3]);
+          }
         }
       }
+      if (st + 1 < o_stages) store_o(st + 1);
       __syncthreads();
     }
     const float dl = inv_s[wr + g], dh = inv_s[wr + g + 8];
@@ -680,28 +756,26 @@ int lt_mlstm_prefill(const void* q, const void* k, const void* v, long long ld, 
   if (N == 0) return 0;
   const int chunks = (N + kMlChunk - 1) / kMlChunk;
   const size_t smem_out = mlstm_out_smem(D);
-  const size_t smem_state = size_t(3) * kMlChunk * kMlPitch * 2;
+  const size_t smem_state = kMlStateSmem;
   const size_t smem_scan = size_t(chunks) * 4;
-  const int dt = (D + kMlRows - 1) / kMlRows, et = (E + kMlRows - 1) / kMlRows;
-  if (smem_out > 220 * 1024 || H > 65535 || dt * et > 65535 || smem_scan > 200 * 1024) return -4;
+  const int dt = (D + kMlRows - 1) / kMlRows;
+  if (smem_out > 220 * 1024 || H > 65535 || dt > 65535 || 2 * smem_scan > 48 * 1024) return -4;      // 6144 chunks: 786432 tokens at a time
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const int aligned = ld % 8 == 0 && D % 8 == 0 && E % 8 == 0 && al(q) && al(k) && al(v);
   const int bank = start & 1, bank1 = (start + N) & 1, fresh = start == 0;
-  mlstm_gates_kernel<<<H, 256, 0, st>>>(logits, ib, fb, cap, fresh ? nullptr : m + (long long)bank * H, a, f, cmax, m_start, N, H, chunks);
+  mlstm_gates_kernel<<<H, 256, 2 * smem_scan, st>>>(logits, ib, fb, cap, fresh ? nullptr : m + (long long)bank * H, a, f, cmax, m_start, N, H, chunks);
   LT_LAUNCH_CHECK();
   LT_RETURN_IF_CUDA(cudaFuncSetAttribute(mlstm_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_state)));
-  mlstm_chunk_state_kernel<<<dim3(chunks, H, dt * et), 128, smem_state, st>>>(
+  mlstm_chunk_state_kernel<<<dim3(chunks, H, dt), 256, smem_state, st>>>(
       static_cast<const __nv_bfloat16*>(k), static_cast<const __nv_bfloat16*>(v), ld, a, cmax, m_start, U, nU, N, D, E, chunks, aligned);
   LT_LAUNCH_CHECK();
-  const bool v4 = ((long long)D * E) % 4 == 0;
+  const bool v4 = D % 4 == 0;                 // then D E and every offset are multiples of 4 too
   const long long per = v4 ? 1024 : 256;
-  const unsigned sb = unsigned(((long long)D * E + D + per - 1) / per);
+  const unsigned sb = unsigned(((long long)D * E + per - 1) / per + (D + per - 1) / per);
   if (v4) {
-    if (smem_scan > 48 * 1024) LT_RETURN_IF_CUDA(cudaFuncSetAttribute(mlstm_chunk_scan_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_scan)));
     mlstm_chunk_scan_kernel<4><<<dim3(sb, H), 256, smem_scan, st>>>(U, nU, cmax, m_start, S, n + (long long)bank * H * D, n + (long long)bank1 * H * D, m + (long long)bank1 * H, N, D, E, chunks, fresh);
   } else {
-    if (smem_scan > 48 * 1024) LT_RETURN_IF_CUDA(cudaFuncSetAttribute(mlstm_chunk_scan_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem_scan)));
     mlstm_chunk_scan_kernel<1><<<dim3(sb, H), 256, smem_scan, st>>>(U, nU, cmax, m_start, S, n + (long long)bank * H * D, n + (long long)bank1 * H * D, m + (long long)bank1 * H, N, D, E, chunks, fresh);
   }
   LT_LAUNCH_CHECK();

@@ -32,30 +32,52 @@ struct QkvParams {
   void* v_lin;
 };
 
-template <typename T>
-__global__ void __launch_bounds__(128) qkv_rope_kernel(const QkvParams p) {
-  extern __shared__ float2 cs[];         // [rot_dims / 2] (cos, sin) of this token
+constexpr int kQkvThreads = 256;
+// V: elements per access of the projection row (8: bf16 in 16-byte pieces; segment offsets and sizes are multiples of it).
+template <typename T, int V>
+__global__ void __launch_bounds__(kQkvThreads) qkv_rope_kernel(const QkvParams p) {
+  extern __shared__ float2 cs[];         // [rot_dims / 2] (cos, sin) of this token, then the row: q, k, v as fp32
   __shared__ float red[64];
+  float* q_s = reinterpret_cast<float*>(cs + p.rot_dims / 2);
+  const int nq = p.H * p.D, nk = p.G * p.D, nv = p.G * p.E;
+  float* k_s = q_s + nq;
+  float* v_s = k_s + nk;
   const int n = blockIdx.x;
   const T* row = static_cast<const T*>(p.proj) + n * p.ld;
   const int pos = p.positions[n], slot = p.slots[n];
-  for (int i = threadIdx.x; i < p.rot_dims / 2; i += blockDim.x) {
+  float sum[2] = {0.f, 0.f};
+  auto fetch = [&](const T* src, float* dst, int count, float& acc) {
+    for (int i = threadIdx.x * V; i < count; i += kQkvThreads * V) {
+      if constexpr (V == 8) {
+        const float4 a = ldf4(src + i), b = ldf4(src + i + 4);
+        *reinterpret_cast<float4*>(dst + i) = a;
+        *reinterpret_cast<float4*>(dst + i + 4) = b;
+        acc += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w + b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+      } else {
+        const float f = ldf(src + i);
+        dst[i] = f;
+        acc += f * f;
+      }
+    }
+  };
+  float unused = 0.f;
+  fetch(row + p.q_off, q_s, nq, sum[0]);
+  fetch(row + p.k_off, k_s, nk, sum[1]);
+  fetch(row + p.v_off, v_s, nv, unused);
+  for (int i = threadIdx.x; i < p.rot_dims / 2; i += kQkvThreads) {
     // the angle can be far outside a period: reduce it in double before the fp32 sine
     const double turns = double(pos) * p.freq[i] * 0.15915494309189535;
     float s, c;
     sincospif(float(2.0 * (turns - rint(turns))), &s, &c);
     cs[i] = make_float2(c * p.gain, s * p.gain);
   }
-  float a = 0.f, b = 0.f;
-  if (p.q_norm) for (int i = threadIdx.x; i < p.H * p.D; i += blockDim.x) { const float f = ldf(row + p.q_off + i); a += f * f; }
-  if (p.k_norm) for (int i = threadIdx.x; i < p.G * p.D; i += blockDim.x) { const float f = ldf(row + p.k_off + i); b += f * f; }
-  const float2 s2 = block_sum2(a, b, red);          // also publishes cs
-  const float rq = p.q_norm ? 1.f / sqrtf(s2.x / (p.H * p.D) + p.eps) : 1.f;
-  const float rk = p.k_norm ? 1.f / sqrtf(s2.y / (p.G * p.D) + p.eps) : 1.f;
-  // pairs (d, d + 1) of one head of q or k
-  auto pair = [&](const T* src, const float* w, int h, int d, float r) -> float2 {
+  const float2 s2 = block_sum2(sum[0], sum[1], red);          // also publishes the row and the angles
+  const float rq = p.q_norm ? 1.f / sqrtf(s2.x / nq + p.eps) : 1.f;
+  const float rk = p.k_norm ? 1.f / sqrtf(s2.y / nk + p.eps) : 1.f;
+  // the pair (d, d + 1) of one head of q or k
+  auto pair = [&](const float* src, const float* w, int h, int d, float r) -> float2 {
     const int c = h * p.D + d;
-    float u = d < p.D ? ldf(src + c) * r : 0.f, v = d + 1 < p.D ? ldf(src + c + 1) * r : 0.f;
+    float u = d < p.D ? src[c] * r : 0.f, v = d + 1 < p.D ? src[c + 1] * r : 0.f;
     if (w) {
       if (d < p.D) u *= w[c];
       if (d + 1 < p.D) v *= w[c + 1];
@@ -66,31 +88,28 @@ __global__ void __launch_bounds__(128) qkv_rope_kernel(const QkvParams p) {
     }
     return make_float2(u, v);
   };
+  const int dq = p.DP / 4;                  // DP and EP are multiples of 8
   T* q_out = static_cast<T*>(p.q_out) + (long long)n * p.H * p.DP;
-  for (int i = threadIdx.x; i < p.H * (p.DP / 2); i += blockDim.x) {
-    const int h = i / (p.DP / 2), d = (i % (p.DP / 2)) * 2;
-    const float2 f = pair(row + p.q_off, p.q_norm, h, d, rq);
-    stf(q_out + h * p.DP + d, f.x);
-    stf(q_out + h * p.DP + d + 1, f.y);
+  for (int i = threadIdx.x; i < p.H * dq; i += kQkvThreads) {
+    const int h = i / dq, d = (i % dq) * 4;
+    const float2 a = pair(q_s, p.q_norm, h, d, rq), b = pair(q_s, p.q_norm, h, d + 2, rq);
+    stf4(q_out + h * p.DP + d, make_float4(a.x, a.y, b.x, b.y));
   }
   const int blk = slot / p.block_size, off = slot % p.block_size;
-  for (int i = threadIdx.x; i < p.G * (p.DP / 2); i += blockDim.x) {
-    const int g = i / (p.DP / 2), d = (i % (p.DP / 2)) * 2;
-    const float2 f = pair(row + p.k_off, p.k_norm, g, d, rk);
-    T* dst = static_cast<T*>(p.k_cache) + (((long long)blk * p.G + g) * p.block_size + off) * p.DP + d;
-    stf(dst, f.x);
-    stf(dst + 1, f.y);
-    if (p.k_lin) {
-      T* lin = static_cast<T*>(p.k_lin) + ((long long)n * p.G + g) * p.DP + d;
-      stf(lin, f.x);
-      stf(lin + 1, f.y);
-    }
+  for (int i = threadIdx.x; i < p.G * dq; i += kQkvThreads) {
+    const int g = i / dq, d = (i % dq) * 4;
+    const float2 a = pair(k_s, p.k_norm, g, d, rk), b = pair(k_s, p.k_norm, g, d + 2, rk);
+    const float4 f = make_float4(a.x, a.y, b.x, b.y);
+    stf4(static_cast<T*>(p.k_cache) + (((long long)blk * p.G + g) * p.block_size + off) * p.DP + d, f);
+    if (p.k_lin) stf4(static_cast<T*>(p.k_lin) + ((long long)n * p.G + g) * p.DP + d, f);
   }
-  for (int i = threadIdx.x; i < p.G * p.EP; i += blockDim.x) {
-    const int g = i / p.EP, e = i % p.EP;
-    const float f = e < p.E ? ldf(row + p.v_off + g * p.E + e) : 0.f;
-    stf(static_cast<T*>(p.v_cache) + (((long long)blk * p.G + g) * p.block_size + off) * p.EP + e, f);
-    if (p.v_lin) stf(static_cast<T*>(p.v_lin) + ((long long)n * p.G + g) * p.EP + e, f);
+  const int eq = p.EP / 4;
+  for (int i = threadIdx.x; i < p.G * eq; i += kQkvThreads) {
+    const int g = i / eq, e = (i % eq) * 4;
+    const float* v = v_s + g * p.E;
+    const float4 f = make_float4(e < p.E ? v[e] : 0.f, e + 1 < p.E ? v[e + 1] : 0.f, e + 2 < p.E ? v[e + 2] : 0.f, e + 3 < p.E ? v[e + 3] : 0.f);
+    stf4(static_cast<T*>(p.v_cache) + (((long long)blk * p.G + g) * p.block_size + off) * p.EP + e, f);
+    if (p.v_lin) stf4(static_cast<T*>(p.v_lin) + ((long long)n * p.G + g) * p.EP + e, f);
   }
 }
 
@@ -215,13 +234,16 @@ int lt_qkv_rope(int fp32, const void* proj, long long ld, int n, int q_off, int 
                 void* k_lin, void* v_lin, void* stream) {
   using namespace lt;
   if (n == 0) return 0;
-  if (G < 1 || H % G != 0 || DP < D || EP < E || (DP & 1) || rot_dims > D || (rot_dims & 1) || rot_dims > 8192) return -4;
+  const long long smem = (long long)rot_dims * 4 + ((long long)H * D + (long long)G * (D + E)) * 4;
+  if (G < 1 || H % G != 0 || DP < D || EP < E || (DP & 7) || (EP & 7) || rot_dims > D || (rot_dims & 1) || smem > 220 * 1024) return -4;
   QkvParams p{proj, ld, q_off, k_off, v_off, H, G, D, E, DP, EP, q_norm, k_norm, eps, positions, slots, freq, rot_dims, gain,
               q_out, k_cache, v_cache, block_size, k_lin, v_lin};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int smem = rot_dims * 4 + 16;
-  if (fp32) qkv_rope_kernel<float><<<n, 128, smem, st>>>(p);
-  else qkv_rope_kernel<__nv_bfloat16><<<n, 128, smem, st>>>(p);
+  const bool v8 = !fp32 && ((ld | q_off | k_off | v_off | (H * D) | (G * D) | (G * E)) & 7) == 0 && (rot_dims & 3) == 0 &&
+                  (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
+  auto kern = fp32 ? qkv_rope_kernel<float, 1> : v8 ? qkv_rope_kernel<__nv_bfloat16, 8> : qkv_rope_kernel<__nv_bfloat16, 1>;
+  if (smem > 48 * 1024) LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+  kern<<<n, kQkvThreads, smem, st>>>(p);
   LT_LAUNCH_CHECK();
   return 0;
 }

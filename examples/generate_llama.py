@@ -1,5 +1,5 @@
-"""Text generation from a Hugging Face Llama directory (config.json + *.safetensors) on the serving path of this package:
-weights converted by `models.llama_io`, continuous batching over a paged KV cache, CUDA-graph decode steps.
+"""Text generation from a model directory (config.json + *.safetensors: a Hugging Face Llama, a Safuvik, any family of
+`models.registry`) on the serving path of this package: continuous batching over a paged KV cache, CUDA-graph decode steps.
 
     python examples/generate_llama.py --model /models/llama --sentencepiece /models/llama/tokenizer.model \
         --prompt "The capital of France is" --prompt "Once upon a time" --max-new-tokens 64 --temperature 0.8 --top-p 0.95
@@ -17,8 +17,8 @@ sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
 import torch
 
-from litetorch_b200.models import llama_io
-from litetorch_b200.models.llama_serving import generate
+from litetorch_b200.models import registry
+from litetorch_b200.models.serving_base import generate
 
 
 def main(argv=None) -> dict:
@@ -35,6 +35,7 @@ def main(argv=None) -> dict:
     ap.add_argument("--seed", type=int, default=0)
     ap.add_argument("--eos-id", type=int, default=-1)
     ap.add_argument("--device", default="cuda")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="precision on a GPU, where the family has both")
     args = ap.parse_args(argv)
     if args.sentencepiece:
         import sentencepiece as spm
@@ -49,13 +50,7 @@ def main(argv=None) -> dict:
         encode = lambda s: [int(t) for t in s.split(",")]
         decode = lambda ids: ",".join(str(i) for i in ids)
         eos = args.eos_id
-    kw = {}
-    if args.device == "cpu":
-        from litetorch_b200.models.llama import LocalWeights
-        with open(os.path.join(args.model, "config.json")) as f:
-            cfg = llama_io.config_from_hf(json.load(f))
-        kw["weights"] = LocalWeights(cfg, "cpu", seed=0, param_dtype=torch.float32)
-    engine = llama_io.load_pretrained(args.model, device=args.device, **kw)
+    engine = registry.load_engine(args.model, args.device, getattr(torch, args.dtype))
     prompts = [encode(p) for p in args.prompt]
     t0 = time.time()
     outs = generate(engine, prompts, args.max_new_tokens, temperature=args.temperature, top_k=args.top_k, top_p=args.top_p,

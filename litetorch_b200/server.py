@@ -229,32 +229,24 @@ def tokenizer(sentencepiece: str = "", byte_level: bool = False):
 
 def main(argv=None):
     import torch
-    from .models import llama_io
-    from .models.llama_serving import LlamaKVModel
+    from .models import registry
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", required=True, help="Hugging Face directory (config.json + *.safetensors)")
+    ap.add_argument("--model", required=True, help="model directory (config.json + *.safetensors) of any registered family")
     ap.add_argument("--host", default="127.0.0.1")
     ap.add_argument("--port", type=int, default=8000)
     ap.add_argument("--sentencepiece", default="")
     ap.add_argument("--bytes", action="store_true")
     ap.add_argument("--device", default="cuda")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="precision on a GPU, where the family has both")
     ap.add_argument("--kv-blocks", type=int, default=4096)
     ap.add_argument("--block-size", type=int, default=16)
     ap.add_argument("--max-num-seqs", type=int, default=64)
     ap.add_argument("--max-batched-tokens", type=int, default=4096)
     ap.add_argument("--prefix-cache-mb", type=int, default=0, help="keep K / V of finished prompts for reuse by prompts that share a prefix")
     args = ap.parse_args(argv)
-    kw = {}
-    if args.device == "cpu":
-        import os
-        from .models.llama import LocalWeights
-        with open(os.path.join(args.model, "config.json")) as f:
-            cfg = llama_io.config_from_hf(json.load(f))
-        kw["weights"] = LocalWeights(cfg, "cpu", seed=0, param_dtype=torch.float32)
-    engine = llama_io.load_pretrained(args.model, device=args.device, **kw)
-    model = LlamaKVModel(engine, num_blocks=args.kv_blocks, block_size=args.block_size,
-                         kv_dtype=torch.float32 if args.device == "cpu" else torch.bfloat16,
-                         prefix_cache_bytes=args.prefix_cache_mb << 20)
+    engine = registry.load_engine(args.model, args.device, getattr(torch, args.dtype))
+    model = registry.new_serving(engine, num_blocks=args.kv_blocks, block_size=args.block_size, max_num_seqs=args.max_num_seqs,
+                                 prefix_cache_bytes=args.prefix_cache_mb << 20)
     encode, decode, eos = tokenizer(args.sentencepiece, args.bytes)
     loop = EngineLoop(model, args.kv_blocks, args.block_size, args.max_num_seqs, args.max_batched_tokens, eos_id=eos,
                       max_context=engine.cfg.max_seq)

@@ -17,31 +17,15 @@ import json
 import torch
 
 
-def main():
-    ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="llama-1.1b", choices=["llama-1.1b", "llama-tiny", "llama3-8b"])
-    ap.add_argument("--batches", default="1,32,128")
-    ap.add_argument("--contexts", default="2048,16384")
-    ap.add_argument("--no-graphs", action="store_true", help="launch every kernel of a step instead of replaying a CUDA graph")
-    ap.add_argument("--hbm-gbs", type=float, default=6552.0, help="measured copy bandwidth used as the roofline denominator")
-    a = ap.parse_args()
-    from ..models.llama import LlamaConfig, LlamaEngine
-    from ..models.llama_serving import LlamaKVModel
-    from ..ops import kernels as K
-    cfg = {"llama-1.1b": LlamaConfig.llama_1b, "llama-tiny": LlamaConfig.tiny, "llama3-8b": LlamaConfig.llama3_8b}[a.model]()
-    batches = [int(x) for x in a.batches.split(",")]
-    contexts = [int(x) for x in a.contexts.split(",")]
-    import dataclasses
-    cfg = dataclasses.replace(cfg, max_seq=max(contexts) + 64)
+def inference_engine(cfg):
+    """A Llama engine with random bf16 weights alone (no gradients, no optimizer state)."""
+    import math
+
+    from ..models.llama import LlamaEngine, LocalWeights, kernels_for, param_specs, rope_tables
     dev = torch.device("cuda")
-    # inference only: the bf16 parameters alone (no gradients, no optimizer state)
-    eng = LlamaEngine.__new__(LlamaEngine)
-    from ..models.llama import LocalWeights, kernels_for, rope_tables
 
     class _InferenceWeights(LocalWeights):
         def __init__(self, cfg, device, seed):
-            from ..models.llama import param_specs
-            import math
             self.cfg, self.K = cfg, kernels_for(device)
             self.specs = param_specs(cfg)
             self.by_name = {s.name: s for s in self.specs}
@@ -53,9 +37,30 @@ def main():
             self.flat_p[:self.n_matrix].normal_(0.0, cfg.init_std, generator=torch.Generator(device=device).manual_seed(seed))
             self.flat_p[self.n_matrix:].fill_(1.0)
 
+    eng = LlamaEngine.__new__(LlamaEngine)
     eng.cfg, eng.device, eng.K = cfg, dev, kernels_for(dev)
     eng.w = _InferenceWeights(cfg, dev, 0)
     eng.cos, eng.sin = rope_tables(cfg, dev)
+    return eng
+
+
+def main():
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--model", default="llama-1.1b", choices=["llama-1.1b", "llama-tiny", "llama3-8b"])
+    ap.add_argument("--batches", default="1,32,128")
+    ap.add_argument("--contexts", default="2048,16384")
+    ap.add_argument("--no-graphs", action="store_true", help="launch every kernel of a step instead of replaying a CUDA graph")
+    ap.add_argument("--hbm-gbs", type=float, default=6552.0, help="measured copy bandwidth used as the roofline denominator")
+    a = ap.parse_args()
+    from ..models.llama import LlamaConfig
+    from ..models.llama_serving import LlamaKVModel
+    from ..ops import kernels as K
+    cfg = {"llama-1.1b": LlamaConfig.llama_1b, "llama-tiny": LlamaConfig.tiny, "llama3-8b": LlamaConfig.llama3_8b}[a.model]()
+    batches = [int(x) for x in a.batches.split(",")]
+    contexts = [int(x) for x in a.contexts.split(",")]
+    import dataclasses
+    cfg = dataclasses.replace(cfg, max_seq=max(contexts) + 64)
+    eng = inference_engine(cfg)
     weight_bytes = eng.w.n_matrix * 2 - cfg.vocab_size * cfg.d_model * 2          # the embedding table is only gathered from
     bs = 16
     rows = []
