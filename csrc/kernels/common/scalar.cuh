@@ -42,6 +42,43 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// Sums of N (a power of two up to 32) values over the warp with N - 1 + log2(32 / N) exchanges instead of 5 N: lane l gets
+// the sum of value l % N.  v is used up.
+template <int N>
+__device__ __forceinline__ float warp_sum_each(float (&v)[N]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int half = N / 2; half >= 1; half >>= 1) {
+    const bool up = (lane & half) != 0;
+#pragma unroll
+    for (int i = 0; i < half; ++i) {
+      const float keep = up ? v[i + half] : v[i], give = up ? v[i] : v[i + half];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, half);
+    }
+  }
+  float r = v[0];
+#pragma unroll
+  for (int o = N; o < 32; o <<= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+  return r;
+}
+
+// Eight neighbouring elements as fp32; p is aligned to eight elements.
+__device__ __forceinline__ void ldf8(const float* p, float (&v)[8]) {
+  const float4 a = ldf4(p), b = ldf4(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void ldf8(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 f = __bfloat1622float2(h[i]);
+    v[2 * i] = f.x;
+    v[2 * i + 1] = f.y;
+  }
+}
+
 // Sums of two values over the block, returned to every thread; red holds 64 floats and is free again on return.
 __device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;

@@ -57,57 +57,44 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, TO* __restric
     }
 }
 
-// y[R, J] (fp32) = x[R, K] @ w[J, K]^T for a narrow w: a CTA makes a 4 x 4 patch, its eight warps share K (so that a
+// y[R, J] (fp32) = x[R, K] @ w[J, K]^T for a narrow w: a CTA makes a 4 x 8 patch, its eight warps share K (so that a
 // handful of rows is not bound by the latency of one long walk) and fold their sums through shared memory.
-constexpr int kRdTile = 4;
+constexpr int kRdR = 4, kRdJ = 8;
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
 rows_dot_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, float* __restrict__ y, int R, int J, int K) {
-  __shared__ float part[8][kRdTile * kRdTile];
+  __shared__ float part[8][kRdR * kRdJ];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int r0 = blockIdx.x * kRdTile, j0 = blockIdx.y * kRdTile;
-  const T* xp[kRdTile];
-  const T* wp[kRdTile];
-#pragma unroll
-  for (int i = 0; i < kRdTile; ++i) {            // rows past the end read the last row; their results are dropped
-    xp[i] = x + min(r0 + i, R - 1) * ldx;
-    wp[i] = w + (long long)min(j0 + i, J - 1) * K;
-  }
-  float acc[kRdTile][kRdTile] = {};
-#pragma unroll 2
+  const int r0 = blockIdx.x * kRdR, j0 = blockIdx.y * kRdJ;
+  float acc[kRdR * kRdJ] = {};
   for (int k = threadIdx.x * V; k < K; k += 256 * V) {
-    float xv[kRdTile][V], wv[kRdTile][V];
+    float xv[kRdR][V];
+    // rows past the end read the last row; their results are dropped
 #pragma unroll
-    for (int i = 0; i < kRdTile; ++i) {
-      if constexpr (V == 4) {
-        const float4 a = ldf4(xp[i] + k), b = ldf4(wp[i] + k);
-        xv[i][0] = a.x; xv[i][1] = a.y; xv[i][2] = a.z; xv[i][3] = a.w;
-        wv[i][0] = b.x; wv[i][1] = b.y; wv[i][2] = b.z; wv[i][3] = b.w;
-      } else {
-        xv[i][0] = ldf(xp[i] + k);
-        wv[i][0] = ldf(wp[i] + k);
-      }
+    for (int i = 0; i < kRdR; ++i) {
+      const T* src = x + min(r0 + i, R - 1) * ldx + k;
+      if constexpr (V == 8) ldf8(src, xv[i]);
+      else xv[i][0] = ldf(src);
     }
 #pragma unroll
-    for (int r = 0; r < kRdTile; ++r)
+    for (int c = 0; c < kRdJ; ++c) {
+      const T* src = w + (long long)min(j0 + c, J - 1) * K + k;
+      float wv[V];
+      if constexpr (V == 8) ldf8(src, wv);
+      else wv[0] = ldf(src);
 #pragma unroll
-      for (int c = 0; c < kRdTile; ++c)
+      for (int r = 0; r < kRdR; ++r)
 #pragma unroll
-        for (int v = 0; v < V; ++v) acc[r][c] = fmaf(xv[r][v], wv[c][v], acc[r][c]);
+        for (int v = 0; v < V; ++v) acc[r * kRdJ + c] = fmaf(xv[r][v], wv[v], acc[r * kRdJ + c]);
+    }
   }
-#pragma unroll
-  for (int r = 0; r < kRdTile; ++r)
-#pragma unroll
-    for (int c = 0; c < kRdTile; ++c) {
-      const float v = warp_sum(acc[r][c]);
-      if (lane == 0) part[warp][r * kRdTile + c] = v;
-    }
+  part[warp][lane] = warp_sum_each<kRdR * kRdJ>(acc);
   __syncthreads();
-  if (threadIdx.x < kRdTile * kRdTile) {
-    const int r = r0 + threadIdx.x / kRdTile, c = j0 + threadIdx.x % kRdTile;
+  if (warp == 0) {
+    const int r = r0 + lane / kRdJ, c = j0 + lane % kRdJ;
     float v = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v += part[i][threadIdx.x];
+    for (int i = 0; i < 8; ++i) v += part[i][lane];
     if (r < R && c < J) y[(long long)r * J + c] = v;
   }
 }
@@ -140,14 +127,14 @@ int lt_gemm_simt(int in_fp32, int out_fp32, const void* A, const void* B, void* 
 int lt_rows_dot(int fp32, const void* x, long long ldx, const void* w, float* y, int R, int J, int K, void* stream) {
   using namespace lt;
   if (R <= 0 || J <= 0) return 0;
-  dim3 grid((R + kRdTile - 1) / kRdTile, (J + kRdTile - 1) / kRdTile);
+  dim3 grid((R + kRdR - 1) / kRdR, (J + kRdJ - 1) / kRdJ);
   if (grid.y > 65535) return -4;
-  const bool v4 = K % 4 == 0 && ldx % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
+  const bool v8 = K % 8 == 0 && ldx % 8 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   using bf = __nv_bfloat16;
 #define LT_RD(T, V) rows_dot_kernel<T, V><<<grid, 256, 0, st>>>(static_cast<const T*>(x), ldx, static_cast<const T*>(w), y, R, J, K)
-  if (fp32) { if (v4) LT_RD(float, 4); else LT_RD(float, 1); }
-  else { if (v4) LT_RD(bf, 4); else LT_RD(bf, 1); }
+  if (fp32) { if (v8) LT_RD(float, 8); else LT_RD(float, 1); }
+  else { if (v8) LT_RD(bf, 8); else LT_RD(bf, 1); }
 #undef LT_RD
   LT_LAUNCH_CHECK();
   return 0;

@@ -52,6 +52,26 @@ static int launch_gemm_pair(const CUtensorMap& tmA, const CUtensorMap& tmB, cons
   return 0;
 }
 
+template <int BLOCK_N>
+__global__ void __launch_bounds__(kGemmThreads, 1)
+gemm_block_diag_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const GemmParams p) {
+  gemm_body<BLOCK_N, 0, 0, 0, true>(&tmA, &tmB, p, NoGate(), NoDone());
+}
+
+template <int BLOCK_N>
+static int launch_block_diag(const CUtensorMap& tmA, const CUtensorMap& tmB, const GemmParams& p, int grid, cudaStream_t st) {
+  using Cfg = GemmCfg<BLOCK_N>;
+  auto kern = gemm_block_diag_kernel<BLOCK_N>;
+  static bool configured = false;
+  if (!configured) {
+    LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    configured = true;
+  }
+  kern<<<grid, kGemmThreads, Cfg::kSmemBytes, st>>>(tmA, tmB, p);
+  LT_LAUNCH_CHECK();
+  return 0;
+}
+
 // 0: never use CTA pairs; 1: where the cost model prefers them; 2: wherever the shape allows.
 static std::atomic<int> g_pair_mode{1};
 int gemm_pair_mode() { return g_pair_mode.load(); }
@@ -172,7 +192,7 @@ int lt_gemm_block_diag(const void* A, const void* B, float* C, int M, int blocks
                        void* stream) {
   using namespace lt;
   if (M <= 0 || blocks <= 0) return 0;
-  if ((K & 7) || nb % 128 != 0 || (lda & 7) || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15))
+  if ((K & 7) || nb % 128 != 0 || (lda & 7) || (ldc & 3) || (reinterpret_cast<uintptr_t>(C) & 15) || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15))
     return -int(kStatusBadArgument);
   const int block_n = nb % 256 == 0 ? 256 : 128;
   GemmParams p{};
@@ -189,7 +209,7 @@ int lt_gemm_block_diag(const void* A, const void* B, float* C, int M, int blocks
   int grid = sm_count();
   if (grid > p.num_tiles) grid = p.num_tiles;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return block_n == 256 ? launch_gemm<256, 0, 0>(tmA, tmB, p, grid, st) : launch_gemm<128, 0, 0>(tmA, tmB, p, grid, st);
+  return block_n == 256 ? launch_block_diag<256>(tmA, tmB, p, grid, st) : launch_block_diag<128>(tmA, tmB, p, grid, st);
 }
 
 static int gemm_launch(int kind, const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,

@@ -287,6 +287,36 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, int ro
   }
 }
 
+// 32 rows x 32 columns of fp32 results, one row per lane, to global memory in whole 128-byte lines: eight lanes exchange
+// their 16-byte pieces until each of them holds the same column piece of eight rows, so that a store instruction covers four
+// full lines instead of 32 fragments.  All 32 lanes take part; columns are inside the matrix, rows are checked.
+__device__ __forceinline__ void store_f32_lines(const GemmParams& p, int row, int col0, uint32_t (&r)[32]) {
+  const int l = lane_id() & 7;
+#pragma unroll
+  for (int half = 4; half >= 1; half >>= 1) {
+    const bool up = (l & half) != 0;
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      if (u & half) continue;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        uint32_t& a = r[u * 4 + w];
+        uint32_t& b = r[(u + half) * 4 + w];
+        const uint32_t got = __shfl_xor_sync(0xffffffffu, up ? a : b, half);
+        if (up) a = got;
+        else b = got;
+      }
+    }
+  }
+  // piece u now belongs to the u-th row of this group of eight, columns 4 l .. 4 l + 3
+  float* base = static_cast<float*>(p.C) + (long long)(row - l) * p.ldc + col0 + l * 4;
+#pragma unroll
+  for (int u = 0; u < 8; ++u)
+    if (row - l + u < p.M)
+      *reinterpret_cast<uint4*>(base + (long long)u * p.ldc) = make_uint4(r[u * 4], r[u * 4 + 1], r[u * 4 + 2], r[u * 4 + 3]);
+}
+
+
 // The body shared by all GEMM kernels. `gate(m_blk, n_blk, kb, status)` is called by the producer
 // before it loads k-block kb of a tile and returns false if a bounded wait ran out; `done(m_blk, n_blk)`
 // is called by one thread of each epilogue warp after the warp's rows of a tile are in global memory.
@@ -294,7 +324,8 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, int ro
 // format bits of the run-time instruction descriptor), 2 = kind::tf32, 3 = kind::i8, 4 = kind::f8f6f4 with e4m3 operands.  It is a template parameter and
 // not a run-time branch on purpose: a kernel that contains tcgen05.mma instructions of more than one kind ran its
 // bf16 MMAs at half rate (measured: 1000 instead of 512 cycles per 256 x 256 x 64 block with no loads in flight).
-template <int BLOCK_N, int A_MAJOR, int B_MAJOR, int MMA_KIND = 0, class TileGate, class TileDone>
+// DIAG: the block-diagonal product (GemmParams::diag_n) with fp32 results and nothing else in the epilogue.
+template <int BLOCK_N, int A_MAJOR, int B_MAJOR, int MMA_KIND = 0, bool DIAG = false, class TileGate, class TileDone>
 __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensorMap* tmB, const GemmParams& p,
                                           TileGate gate, TileDone done, int cta_first = 0) {
   // CTAs [0, cta_first) of the grid belong to another role of a fused kernel; the GEMM uses the rest.
@@ -364,7 +395,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensor
           const uint32_t a_dst = smem_base + stage * Cfg::kStageBytes;
           const uint32_t b_dst = a_dst + Cfg::kABytes;
           if (A_MAJOR == 0) {
-            const int a_off = p.diag_n > 0 ? (n_blk * BLOCK_N / p.diag_n) * p.K : 0;
+            const int a_off = DIAG ? (n_blk * BLOCK_N / p.diag_n) * p.K : 0;
             tma_load_2d(a_dst, tmA, fb, a_off + kb * kBlockK, m_blk * kBlockM);
           } else {
 #pragma unroll
@@ -504,7 +535,8 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensor
           if (c + 1 < BLOCK_N / 32) load_parts(c + 1);
         }
         const int col0 = n_blk * BLOCK_N + c * 32;
-        if (row < p.M && col0 < p.N) epilogue_store_chunk(p, row, col0, r);
+        if constexpr (DIAG) store_f32_lines(p, row, col0, r);
+        else if (row < p.M && col0 < p.N) epilogue_store_chunk(p, row, col0, r);
       }
       done.fence();
       tc_fence_before();

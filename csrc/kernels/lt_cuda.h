@@ -200,17 +200,17 @@ int lt_conv_causal(int fp32, const void* x, long long ldx, const float* xb, cons
                    void* u, int N, int C, int taps, int start, void* stream);
 int lt_rglru_scan(int fp32, const void* u, const float* gates, const float* rb, const float* ib, const float* sp, const void* y,
                   long long ldy, const float* yb, const void* x, long long ldx, const float* xb, float* state, float* ring,
-                  void* out, int N, int C, int bw, int taps, int start, void* stream);
+                  void* out, float* scratch, int N, int C, int bw, int taps, int start, void* stream);
 int lt_rglru_step(int fp32, const void* x, long long ldx, const float* xb, const float* conv_w, const float* conv_b,
                   const void* gates, const float* rb, const float* ib, const float* sp, const void* y, long long ldy,
-                  const float* yb, float* state, float* ring, const int* slots, const int* positions, void* out, int S, int C,
-                  int bw, int taps, void* stream);
+                  const float* yb, float* state, float* ring, const int* slots, const int* positions, void* u, void* out,
+                  int S, int C, int bw, int taps, void* stream);
 
 // ---- mlstm.cu: matrix memory with exponential gates, chunked prompt kernels and decode step
 int lt_mlstm_prefill(const void* q, const void* k, const void* v, long long ld, const float* logits, const float* ib,
                      const float* fb, float cap, float qscale, const float* norm, float eps, const void* gate, long long ldg,
-                     float* S, float* n, float* m, float* a, float* f, float* cmax, float* m_start, float* U, float* nU, float* o,
-                     void* out, int N, int H, int D, int E, int start, void* stream);
+                     float* S, float* n, float* m, float* a, float* f, float* cmax, float* last, float* m_start, float* U, float* nU,
+                     float* o, void* out, int N, int H, int D, int E, int start, void* stream);
 int lt_mlstm_step(int fp32, const void* q, const void* k, const void* v, long long ld, const float* logits, const float* ib,
                   const float* fb, float cap, float qscale, float* S, float* n, float* m, const int* slots, const int* positions,
                   float* o, int rows, int H, int D, int E, int seq_len, int slot, int start, void* stream);

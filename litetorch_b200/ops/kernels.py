@@ -28,9 +28,9 @@ _SIGS = {
     "lt_window_attn": [_i, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _ll] + [_i] * 9 + [_f, _vp],
     "lt_head_gate": [_i, _vp, _vp, _ll, _vp, _ll, _i, _i, _i, _vp],
     "lt_conv_causal": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
-    "lt_rglru_scan": [_i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
-    "lt_rglru_step": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
-    "lt_mlstm_prefill": [_vp, _vp, _vp, _ll, _vp, _vp, _vp, _f, _f, _vp, _f, _vp, _ll] + [_vp] * 11 + [_i] * 5 + [_vp],
+    "lt_rglru_scan": [_i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "lt_rglru_step": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "lt_mlstm_prefill": [_vp, _vp, _vp, _ll, _vp, _vp, _vp, _f, _f, _vp, _f, _vp, _ll] + [_vp] * 12 + [_i] * 5 + [_vp],
     "lt_mlstm_step": [_i, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _vp, _vp] + [_i] * 7 + [_vp],
     "lt_head_norm_gate": [_i, _vp, _vp, _vp, _ll, _vp, _ll, _i, _i, _f, _vp],
     "lt_status_fetch": [],
@@ -109,7 +109,7 @@ _SIGS = {
 _bound = {}
 
 # Kernels launched per native call; `launch_count()` is what bench.py reports as "gpu_launches".
-_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_paged_decode_window": 2, "lt_mlstm_prefill": 4, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
+_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_paged_decode_window": 2, "lt_mlstm_prefill": 4, "lt_rglru_scan": 3, "lt_rglru_step": 2, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
                       "lt_adam_chunk_elems": 0}
 _launches = [0]
 
@@ -925,9 +925,10 @@ def rglru_scan(u, gates, rb, ib, sp, y, yb, x, xb, state, ring, taps: int, start
     N, C = u.shape
     bw = rb.shape[-1]
     out = torch.empty((N, C), dtype=u.dtype, device=u.device)
+    scratch = torch.empty(3 * C * ((N + 31) // 32), dtype=torch.float32, device=u.device)
     rc = _fn("lt_rglru_scan")(_f32(u), u.data_ptr(), gates.data_ptr(), rb.data_ptr(), ib.data_ptr(), sp.data_ptr(), y.data_ptr(), y.stride(0),
-                              yb.data_ptr(), x.data_ptr(), x.stride(0), _p(xb), state.data_ptr(), ring.data_ptr(), out.data_ptr(), N, C, bw,
-                              taps, start, _stream())
+                              yb.data_ptr(), x.data_ptr(), x.stride(0), _p(xb), state.data_ptr(), ring.data_ptr(), out.data_ptr(), scratch.data_ptr(), N,
+                              C, bw, taps, start, _stream())
     _check(rc, "lt_rglru_scan")
     return out
 
@@ -936,11 +937,11 @@ def rglru_step(x, xb, conv_w, conv_b, gates, rb, ib, sp, y, yb, state, ring, slo
     """One token of every sequence: convolution, gates ([blocks, rows of r | rows of i, bw]), recurrence and output branch; row s uses
     state[slots[s]] [C] and ring[slots[s]] [taps, C]."""
     S, C = x.shape
-    out = torch.empty((S, C), dtype=x.dtype, device=x.device)
+    u, out = (torch.empty((S, C), dtype=x.dtype, device=x.device) for _ in range(2))
     rc = _fn("lt_rglru_step")(_f32(x), x.data_ptr(), x.stride(0), _p(xb), conv_w.data_ptr(), conv_b.data_ptr(), gates.data_ptr(),
                               rb.data_ptr(), ib.data_ptr(), sp.data_ptr(), y.data_ptr(), y.stride(0), yb.data_ptr(), state.data_ptr(),
-                              ring.data_ptr(), slots.data_ptr(), positions.data_ptr(), out.data_ptr(), S, C, rb.shape[-1], conv_w.shape[1],
-                              _stream())
+                              ring.data_ptr(), slots.data_ptr(), positions.data_ptr(), u.data_ptr(), out.data_ptr(), S, C, rb.shape[-1],
+                              conv_w.shape[1], _stream())
     _check(rc, "lt_rglru_step")
     return out
 
@@ -960,7 +961,7 @@ def mlstm_prefill(q, k, v, logits, ib, fb, cap: float, norm, eps: float, gate, S
         _check(rc, "lt_mlstm_step")
         return head_norm_gate(o, norm, gate, H, eps)
     chunks = (N + 127) // 128
-    sizes = [H * N, H * N, H * N, H * (chunks + 1), H * chunks * D * E, H * chunks * D, N * H * E]
+    sizes = [H * N, H * N, H * N, 2 * H * chunks, H * (chunks + 1), H * chunks * D * ((E + 7) // 8 * 8), H * chunks * D, N * H * E]
     offs, total = [], 0
     for s in sizes:
         offs.append(total)
