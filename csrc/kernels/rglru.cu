@@ -96,24 +96,24 @@ conv_causal_kernel(const T* __restrict__ x, long long ldx, const float* __restri
 struct RglruGate {
   float a, b;     // S <- a S + b
 };
+// Both forms work from d = 1 - a: where a is close to 1 the state remembers for thousands of tokens, and an a that is wrong in
+// its last place the same way at every token adds up; 1 - d rounds once.  1 - a^2 = d (2 - d) does not cancel.
 // fp32 activations: the library functions.
 __device__ __forceinline__ RglruGate rglru_gate(const float*, float r_logit, float i_logit, float u, float sp) {
-  const float log_a = -8.f * sigmoid_f(r_logit) * sp;
-  // 1 - a^2 without cancellation where a is close to 1
-  return RglruGate{expf(log_a), sqrtf(-expm1f(2.f * log_a)) * sigmoid_f(i_logit) * u};
+  const float d = -expm1f(-8.f * sigmoid_f(r_logit) * sp);
+  return RglruGate{1.f - d, sqrtf(d * (2.f - d)) * sigmoid_f(i_logit) * u};
 }
 __device__ __forceinline__ float gelu_branch(const float*, float z) { return gelu_tanh_f(z); }
 // bf16 activations: the same in fp32 on the fast exponential and divide (a few units in the last place of fp32).
 __device__ __forceinline__ float fast_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 __device__ __forceinline__ RglruGate rglru_gate(const __nv_bfloat16*, float r_logit, float i_logit, float u, float sp) {
-  const float log_a = -8.f * fast_sigmoid(r_logit) * sp;
-  const float a = __expf(log_a), x = -2.f * log_a;
+  const float x = 8.f * fast_sigmoid(r_logit) * sp;                  // -log a
   // 1 - exp(-x): its power series where the difference would cancel
   const float series = x * (1.f - x * (0.5f - x * (1.f / 6 - x * (1.f / 24 - x * (1.f / 120 - x * (1.f / 720))))));
-  const float rest = x < 0.25f ? series : 1.f - a * a;
+  const float d = x < 0.25f ? series : 1.f - __expf(-x);
   float root;
-  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(root) : "f"(rest));
-  return RglruGate{a, root * fast_sigmoid(i_logit) * u};
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(root) : "f"(d * (2.f - d)));
+  return RglruGate{1.f - d, root * fast_sigmoid(i_logit) * u};
 }
 __device__ __forceinline__ float gelu_branch(const __nv_bfloat16*, float z) {
   // (1 + tanh(y)) / 2 is sigmoid(2 y)
