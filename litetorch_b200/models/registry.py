@@ -120,3 +120,27 @@ def _serve_safuvik(engine, num_blocks, block_size, max_num_seqs, kv_dtype, graph
 
 register(ModelFamily("safuvik", lambda c: c.get("architecture") == "Safuvik", _load_safuvik, _is_safuvik_engine, _serve_safuvik,
                      dtypes=(torch.bfloat16, torch.float32), components=("serving", "hybrid")))
+
+
+# ---------------------------------------------------------------------------------------------------- Ravenex
+def _load_ravenex(directory, config, device, dtype):
+    from .ravenex import RavenexEngine
+    return RavenexEngine.from_directory(directory, config, device, dtype)
+
+
+def _is_ravenex_engine(e) -> bool:
+    from .ravenex import RavenexEngine
+    return isinstance(e, RavenexEngine)
+
+
+def _serve_ravenex(engine, num_blocks, block_size, max_num_seqs, kv_dtype, graphs, prefix_cache_bytes):
+    from .ravenex_serving import RavenexModel
+    if prefix_cache_bytes:
+        raise ValueError("prefix reuse keeps keys and values per head; this family caches latents")
+    if kv_dtype is not None and kv_dtype != engine.dtype:
+        raise TypeError("this family keeps its latents in the activations' type (%s)" % engine.dtype)
+    return RavenexModel(engine, num_blocks=num_blocks, block_size=block_size, graphs=graphs)
+
+
+register(ModelFamily("ravenex", lambda c: c.get("architecture") == "Ravenex", _load_ravenex, _is_ravenex_engine, _serve_ravenex,
+                     dtypes=(torch.bfloat16, torch.float32), components=("serving", "hybrid", "latent")))

@@ -18,41 +18,8 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from .llama import kernels_for
-
-
-@dataclass
-class RotaryConfig:
-    """Rotary embedding of the first `dims` dimensions of a head, with YaRN scaling when `factor` is given."""
-    base: float
-    dims: int
-    factor: Optional[float] = None
-    original: float = 0.0
-    fast: float = 0.0
-    slow: float = 0.0
-
-    @staticmethod
-    def parse(c: Optional[dict]) -> "RotaryConfig":
-        if not c:
-            return RotaryConfig(1.0, 0)
-        s = c.get("scaling") or {}
-        return RotaryConfig(float(c["base"]), int(c["dims"]), float(s["factor"]) if s else None, float(s.get("original", 0)),
-                            float(s.get("fast", 0)), float(s.get("slow", 0)))
-
-    def frequencies(self) -> Tuple[List[float], float]:
-        """(angle per token of every pair, gain of cos and sin)."""
-        n = self.dims
-        freq = [self.base ** (-2.0 * i / n) for i in range(n // 2)]
-        if self.factor is None:
-            return freq, 1.0
-
-        def pair_that_turns(times: float) -> float:          # how many turns a pair makes over the original context
-            return n * math.log(self.original / (2.0 * math.pi * times)) / (2.0 * math.log(self.base))
-
-        lo = max(math.floor(pair_that_turns(self.fast)), 0)
-        hi = min(math.ceil(pair_that_turns(self.slow)), n - 1)
-        width = max(hi - lo, 0.001)
-        ramp = [min(max((i - lo) / width, 0.0), 1.0) for i in range(n // 2)]
-        return [f / self.factor * r + f * (1.0 - r) for f, r in zip(freq, ramp)], 0.1 * math.log(self.factor) + 1.0
+from .rotary import RotaryConfig
+from .weights import checked_fetch, stack_rows
 
 
 @dataclass
@@ -192,19 +159,6 @@ def random_tensor(name: str, shape, gen: torch.Generator, device="cpu", dtype=to
     return z.to(dtype)
 
 
-def _pad_rows(ws: List[torch.Tensor]) -> Tuple[torch.Tensor, List[int]]:
-    """Matrices with the same input stacked by rows, every one starting at a multiple of 8 and the whole a multiple of 64
-    rows (zeros between): one product whose columns are aligned for vector loads."""
-    offs, parts, at = [], [], 0
-    for j, w in enumerate(ws):
-        offs.append(at)
-        end = at + w.shape[0]
-        to = (end + 7) // 8 * 8 if j + 1 < len(ws) else (end + 63) // 64 * 64
-        parts.append(torch.nn.functional.pad(w, (0, 0, 0, to - end)))
-        at = to
-    return torch.cat(parts).contiguous(), offs
-
-
 class HyperWeights:
     def __init__(self, get, p: str):
         self.inn, self.out, self.mix = get(p + "in", torch.float32), get(p + "out", torch.float32), get(p + "mix", torch.float32)
@@ -220,7 +174,7 @@ class SafuvikLayer:
         m, x = p + "mix.", cfg.mixer
         if isinstance(x, ParallelConfig):
             l, r = m + "left.", m + "right."
-            self.w_in, self.offs = _pad_rows([get(l + "q"), get(l + "k"), get(l + "v"), get(l + "g"), get(r + "y"), get(r + "x")])
+            self.w_in, self.offs = stack_rows([get(l + "q"), get(l + "k"), get(l + "v"), get(l + "g"), get(r + "y"), get(r + "x")])
             self.q_norm, self.k_norm = get(l + "q.norm", f32), get(l + "k.norm", f32)
             self.left_o, self.left_out = get(l + "o"), get(l + "out", f32)
             freq, self.rot_gain = x.left.rot.frequencies()
@@ -232,7 +186,7 @@ class SafuvikLayer:
             self.decay = torch.nn.functional.softplus(get(r + "lam", torch.float64)).float()
             self.right_o, self.right_out = get(r + "o"), get(r + "out", f32)
         else:
-            self.w_in, self.offs = _pad_rows([get(m + "q"), get(m + "k"), get(m + "v"), get(m + "g")])
+            self.w_in, self.offs = stack_rows([get(m + "q"), get(m + "k"), get(m + "v"), get(m + "g")])
             self.w_if = torch.cat([get(m + "i"), get(m + "f")]).contiguous()
             self.i_b, self.f_b = get(m + "i.b", f32), get(m + "f.b", f32)
             self.head_norm, self.o = get(m + "norm", f32), get(m + "o")
@@ -253,18 +207,7 @@ class SafuvikEngine:
         if dtype not in (torch.bfloat16, torch.float32):
             raise TypeError("weights run in bfloat16 or float32, not %s" % dtype)
         self.K = kernels_for(self.device)
-        shapes = tensor_shapes(cfg)
-        fetch = tensors if callable(tensors) else tensors.__getitem__
-
-        def get(name, as_dtype=None):
-            try:
-                t = fetch(name)
-            except KeyError:
-                raise KeyError("the checkpoint has no tensor %r" % name) from None
-            if tuple(t.shape) != shapes[name]:
-                raise ValueError("%s: the checkpoint gives %s, the configuration expects %s" % (name, tuple(t.shape), shapes[name]))
-            return t.to(self.device).to(as_dtype or dtype).contiguous()
-
+        get = checked_fetch(tensors, tensor_shapes(cfg), self.device, dtype)
         self.embed, self.head = get("embed"), get("head")
         self.final_norm = get("final.norm", torch.float32)
         self.layers = [SafuvikLayer(lay, get, "l%d." % i, self.device) for i, lay in enumerate(cfg.layers)]

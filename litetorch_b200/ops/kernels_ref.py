@@ -339,8 +339,9 @@ def qkv_rope(proj, q_off, k_off, v_off, H, G, D, E, positions, slots, k_cache, v
 def kv_gather(k_cache, v_cache, table, pos0, n, k_lin, v_lin):
     p = torch.arange(pos0, pos0 + n)
     blk, off = table.long()[p // k_cache.shape[2]], p % k_cache.shape[2]
-    k_lin.copy_(k_cache[blk, :, off])
-    v_lin.copy_(v_cache[blk, :, off])
+    k_lin.copy_(k_cache[blk, :, off].view_as(k_lin))
+    if v_cache is not None:
+        v_lin.copy_(v_cache[blk, :, off].view_as(v_lin))
 
 
 def window_attn(q, k_cache, v_cache, tables, positions, *, D, E, window, scale, gate=None):
@@ -444,3 +445,100 @@ def head_norm_gate(o, w, gate, H, eps):
     R, HE = o.shape
     y = _rms(o.view(R, H, HE // H), eps).reshape(R, HE) * w
     return (y * torch.sigmoid(gate.float())).to(gate.dtype)
+
+
+# ------------------------------------------------------------------------------------------------ latent attention, experts
+_ACT = {"gelu": lambda z: torch.nn.functional.gelu(z, approximate="tanh"), "silu": torch.nn.functional.silu}
+
+
+def residual_norm(x, eps, *, dtype, norm=None, mult=1.0, y=None, y_norm=None, experts=None, tokens=None, embed=None, rows=None, write=True):
+    xs = x if embed is None else embed[tokens.long()].float()
+    pick = slice(None) if rows is None else rows.long()
+    xs = xs[pick]
+    add = None if y is None else y[pick].float()
+    if experts is not None:
+        z, slots, weight = experts
+        e = (z[slots.long()[pick]].float() * weight[pick][..., None]).sum(1)
+        add = e if add is None else add + e
+    if add is not None:
+        xs = xs + mult * (add if y_norm is None else _rms(add, eps, y_norm))
+    if write:
+        x.copy_(xs)
+    return (xs if norm is None else _rms(xs, eps, norm)).to(dtype)
+
+
+def latent_rope(proj, H, d, r, rot, positions, slots, *, freq, gain=1.0, c_off=-1, rank=0, c_norm=None, eps=1e-6, cache=None, q_out=None,
+                lin=None):
+    N = proj.shape[0]
+    angle = positions.double()[:, None] * freq[None]
+    c, s = (torch.cos(angle) * gain).float(), (torch.sin(angle) * gain).float()
+
+    def turn(t, c, s):
+        u, v = t[..., 0:rot:2].float(), t[..., 1:rot:2].float()
+        y = torch.zeros(t.shape[:-1] + (r,))
+        if rot:
+            y[..., 0:rot:2], y[..., 1:rot:2] = u * c - v * s, v * c + u * s
+        return y.to(proj.dtype)
+
+    q = turn(proj[:, :H * (d + r)].view(N, H, d + r)[..., d:d + rot], c[:, None], s[:, None])
+    if q_out is None:
+        proj[:, :H * (d + r)].view(N, H, d + r)[..., d:] = q
+    else:
+        q_out[..., q_out.shape[-1] - r:] = q
+    if c_off < 0:
+        return
+    row = torch.zeros(N, cache.shape[-1], dtype=proj.dtype)
+    row[:, :rank] = _rms(proj[:, c_off:c_off + rank].float(), eps, c_norm).to(proj.dtype)
+    row[:, cache.shape[-1] - r:] = turn(proj[:, c_off + rank:c_off + rank + rot], c, s)
+    bs = cache.shape[2]
+    cache[slots.long() // bs, 0, slots.long() % bs] = row
+    if lin is not None:
+        lin.copy_(row)
+
+
+def head_linear(x, w, out=None):
+    y = torch.einsum("nhk,hmk->nhm", x.float(), w.float()).to(x.dtype).contiguous()
+    if out is None:
+        return y
+    out.copy_(y)
+    return out
+
+
+def shared_rope_fwd(q, k, k_rot, v, *, scale, window=0):
+    T, H, d = k.shape
+    kk = torch.cat([k, k_rot[:, None].expand(T, H, k_rot.shape[1])], 2)
+    return flash_fwd(q[None], kk[None], v[None], causal=True, scale=scale, window=window)[0][0]
+
+
+def latent_decode(q, cache, tables, ctx, *, rank, window, scale, max_keys):
+    return window_attn(q, cache, cache, tables, ctx - 1, D=q.shape[2], E=rank, window=window, scale=scale)
+
+
+def act_glu(gu, act):
+    g, u = gu.float().chunk(2, -1)
+    return (_ACT[act](g) * u).to(gu.dtype)
+
+
+def glu_mlp(x, gu, down, act):
+    return linear(act_glu(linear(x, gu), act), down)
+
+
+def moe_route(logits, correction, top):
+    s = torch.sigmoid(logits.float())
+    idx = torch.argsort(s + correction, dim=-1, descending=True, stable=True)[:, :top]
+    return idx.to(torch.int32), s.gather(1, idx)
+
+
+def moe_experts(x, router, correction, top, gu, down, act):
+    idx, weight = moe_route(rows_dot(x, router), correction, top)
+    flat = idx.reshape(-1).long()
+    z = torch.empty(flat.numel(), x.shape[1], dtype=x.dtype)
+    for e in flat.unique().tolist():
+        at = (flat == e).nonzero()[:, 0]
+        z[at] = glu_mlp(x[at // top], gu[e], down[e], act)
+    return z, torch.arange(flat.numel(), dtype=torch.int32).view(-1, top), weight
+
+
+def token_gate(g, tokens, table, off, dim):
+    e = torch.nn.functional.pad(table[tokens.long(), off:off + dim].float(), (0, g.shape[1] - dim))
+    return (_ACT["gelu"](g.float()) * e).to(g.dtype)

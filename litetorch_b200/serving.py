@@ -68,7 +68,7 @@ class PagedKVCache:
     @classmethod
     def per_layer(cls, shapes, num_blocks: int, block_size: int, device="cuda", dtype=torch.bfloat16) -> "PagedKVCache":
         """Layers that differ: `shapes` has (kv heads, key size, value size) of every layer, None for a layer that keeps no
-        keys.  All layers share the block tables."""
+        keys, value size 0 where the values are made from what is kept as keys.  All layers share the block tables."""
         self = cls.__new__(cls)
         self._init(num_blocks, block_size, shapes, device, dtype, 1.0, 1.0)
         return self
@@ -78,7 +78,7 @@ class PagedKVCache:
         self.fp8 = dtype == torch.float8_e4m3fn
         self.k_scale, self.v_scale = k_scale, v_scale
         self.k = [None if s is None else torch.zeros((num_blocks, s[0], block_size, s[1]), dtype=dtype, device=device) for s in shapes]
-        self.v = [None if s is None else torch.zeros((num_blocks, s[0], block_size, s[2]), dtype=dtype, device=device) for s in shapes]
+        self.v = [None if s is None or not s[2] else torch.zeros((num_blocks, s[0], block_size, s[2]), dtype=dtype, device=device) for s in shapes]
 
     @property
     def bytes_per_token(self) -> int:
