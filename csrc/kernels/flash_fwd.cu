@@ -11,6 +11,9 @@
 //                           the exp2 domain, P_j written to shared memory in the swizzled operand layout.
 // The running maximum is updated lazily: O in TMEM is rescaled only when a row's maximum grew by more
 // than 2^8, which keeps exp2 arguments bounded and makes the rescale (tcgen05.ld/st of O) rare.
+// Query / key size D and value size DV may differ, and KV blocks may be 64 keys where a 128-key block of the larger size does
+// not fit in shared memory.  SHARED: the last 64 columns of a key are the same for all heads (a rotated part beside the
+// heads' own unrotated ones) and come from a tensor of their own, so that keys are never put together in memory.
 // Output: O [B, Tq, Hq, D] bf16 and the natural-log LSE [B, Hq, Tq] fp32 for the backward pass.
 #include "lt_cuda.h"
 #include "common/host.h"
@@ -57,15 +60,16 @@ __device__ __forceinline__ float ex2_approx_f(float x) {
   return y;
 }
 
-template <int D>
+template <int D, int DV, int BKV>
 struct FaFwdCfg {
   static constexpr int kQBytes = kFaBlockQ * D * 2;
-  static constexpr int kKVBytes = kFaBlockKV * D * 2;
-  static constexpr int kPBytes = kFaBlockQ * kFaBlockKV * 2;
+  static constexpr int kKBytes = BKV * D * 2;
+  static constexpr int kVBytes = BKV * DV * 2;
+  static constexpr int kPBytes = kFaBlockQ * BKV * 2;
   static constexpr int kOffQ = 0;
   static constexpr int kOffK = kQBytes;
-  static constexpr int kOffV = kOffK + 2 * kKVBytes;
-  static constexpr int kOffP = kOffV + 2 * kKVBytes;
+  static constexpr int kOffV = kOffK + 2 * kKBytes;
+  static constexpr int kOffP = kOffV + 2 * kVBytes;
   static constexpr int kOffBar = kOffP + 2 * kPBytes;
   static constexpr int kOffSeg = kOffBar + 224;               // KvSeg table (16 entries) + block count
   static constexpr int kOffX = kOffSeg + kFaMaxSegs * 16 + 16;                 // row statistics exchanged between the two column halves
@@ -74,17 +78,18 @@ struct FaFwdCfg {
   // that the aligned layout lies inside the allocation and reports kStatusBadArgument otherwise.
   static constexpr int kSmemBytes = (kNeeded + 1024 <= 232448) ? kNeeded + 1024 : 232448;
   static constexpr int kTmemCols = 512;
-  // Score buffers of 128 columns: three with head_dim 64, so that S of block j+2 is computed while the softmax of
-  // blocks j and j+1 is still reading theirs; tensor memory only has room for two with head_dim 128.
-  static constexpr int kSBufs = (D == 64) ? 3 : 2;
+  // Score buffers of BKV columns beside the two output accumulators: three where tensor memory has room (head_dim 64, or
+  // 64-key blocks), so that S of block j+2 is computed while the softmax of blocks j and j+1 is still reading theirs; else two.
+  static constexpr int kSBufs = (512 - 2 * DV) / BKV < 3 ? (512 - 2 * DV) / BKV : 3;
   static constexpr int kColS = 0;
-  static constexpr int kColO = kSBufs * 128;   // two accumulators of D columns (KV blocks of even / odd index)
+  static constexpr int kColO = kSBufs * BKV;   // two accumulators of DV columns (KV blocks of even / odd index)
+  static_assert(kNeeded <= 232448 && kSBufs >= 2, "does not fit");
 };
 
-template <int D>
+template <int D, int DV, int BKV, bool SHARED>
 __global__ void __launch_bounds__(kFaThreads, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ KvMaps maps, const FlashFwdParams p) {
-  using Cfg = FaFwdCfg<D>;
+  using Cfg = FaFwdCfg<D, DV, BKV>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sbase = smem_u32(smem);
@@ -133,7 +138,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   if (threadIdx.x == 0) {
     // visible KV blocks as runs: own rank first (local memory), then the other ranks
     const int q_last = q_base + kFaBlockQ - 1;
-    const int nb_all = (p.Tk + kFaBlockKV - 1) / kFaBlockKV;
+    const int nb_all = (p.Tk + BKV - 1) / BKV;
     int ns = 0, total = 0;
     for (int i = 0; i < p.cp_world; ++i) {
       const int o = (p.cp_rank + i) % p.cp_world;
@@ -144,21 +149,21 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           const int hk = p.Tk / 2;
           kv0 = h2 * hk;
           kbase = h2 == 0 ? o * hk : (2 * p.cp_world - 1 - o) * hk;
-          nb = hk / kFaBlockKV;
+          nb = hk / BKV;
         } else {
           kv0 = 0;
           kbase = p.cp_world > 1 ? o * p.Tk : 0;
           nb = nb_all;
         }
         if (p.causal) {
-          const int vis = q_last < kbase ? 0 : (q_last - kbase) / kFaBlockKV + 1;
+          const int vis = q_last < kbase ? 0 : (q_last - kbase) / BKV + 1;
           nb = nb < vis ? nb : vis;
         }
         if (p.window > 0 && p.cp_world == 1) {
           // blocks that end before the first query's window are skipped
-          const int first = max(0, q_base - p.window + 1) / kFaBlockKV;
-          kv0 += first * kFaBlockKV;
-          kbase += first * kFaBlockKV;
+          const int first = max(0, q_base - p.window + 1) / BKV;
+          kv0 += first * BKV;
+          kbase += first * BKV;
           nb -= first;
         }
         if (nb > 0) {
@@ -178,8 +183,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     int sidx = 0;
     while (sidx < kFaMaxSegs - 1 && j >= segs[sidx].n) { j -= segs[sidx].n; ++sidx; }
     owner = segs[sidx].owner;
-    kv0 = segs[sidx].kv0 + j * kFaBlockKV;
-    kbase = segs[sidx].kbase + j * kFaBlockKV;
+    kv0 = segs[sidx].kv0 + j * BKV;
+    kbase = segs[sidx].kbase + j * BKV;
   };
 
   if (threadIdx.x == 0) {
@@ -220,11 +225,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         int owner, kv0, kbase;
         locate(j, owner, kv0, kbase);
         if (!mbar_wait(k_empty(s), ((j >> 1) & 1) ^ 1u, abort_flag, p.status, kStatusTimeoutEmpty)) return false;
-        mbar_expect_tx(k_full(s), Cfg::kKVBytes);
+        mbar_expect_tx(k_full(s), Cfg::kKBytes);
 #pragma unroll
         for (int c = 0; c < D / 64; ++c)
-          tma_load_4d(sbase + Cfg::kOffK + s * Cfg::kKVBytes + c * (kFaBlockKV * 128), &maps.k[owner], k_full(s), c * 64, hkv,
-                      kv0, b);
+          if (SHARED && c == D / 64 - 1)
+            tma_load_4d(sbase + Cfg::kOffK + s * Cfg::kKBytes + c * (BKV * 128), &maps.k[1], k_full(s), 0, 0, kv0, b);
+          else
+            tma_load_4d(sbase + Cfg::kOffK + s * Cfg::kKBytes + c * (BKV * 128), &maps.k[owner], k_full(s), c * 64, hkv, kv0, b);
         return true;
       };
       bool okp = load_k(0);
@@ -234,10 +241,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         int owner, kv0, kbase;
         locate(j, owner, kv0, kbase);
         if (!mbar_wait(v_empty(s), ((j >> 1) & 1) ^ 1u, abort_flag, p.status, kStatusTimeoutEmpty)) break;
-        mbar_expect_tx(v_full(s), Cfg::kKVBytes);
+        mbar_expect_tx(v_full(s), Cfg::kVBytes);
 #pragma unroll
-        for (int c = 0; c < D / 64; ++c)
-          tma_load_4d(sbase + Cfg::kOffV + s * Cfg::kKVBytes + c * (kFaBlockKV * 128), &maps.v[owner], v_full(s), c * 64, hkv,
+        for (int c = 0; c < DV / 64; ++c)
+          tma_load_4d(sbase + Cfg::kOffV + s * Cfg::kVBytes + c * (BKV * 128), &maps.v[owner], v_full(s), c * 64, hkv,
                       kv0, b);
       }
     }
@@ -247,10 +254,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     // MMAs of a KV block are split over two issuing threads: this one runs the score products as far ahead as the
     // score buffers allow, warp 1 runs the PV products.
     if (lane == 0 && n_blocks > 0) {
-      constexpr uint32_t idesc_s = make_idesc_f16(kFaBlockQ, kFaBlockKV, 1, 0, 0);
+      constexpr uint32_t idesc_s = make_idesc_f16(kFaBlockQ, BKV, 1, 0, 0);
       const uint64_t q_desc = make_smem_desc_sw128(sbase + Cfg::kOffQ, 16, 1024);
       const uint64_t k_desc0 = make_smem_desc_sw128(sbase + Cfg::kOffK, 16, 1024);
-      const uint64_t k_desc1 = make_smem_desc_sw128(sbase + Cfg::kOffK + Cfg::kKVBytes, 16, 1024);
+      const uint64_t k_desc1 = make_smem_desc_sw128(sbase + Cfg::kOffK + Cfg::kKBytes, 16, 1024);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, kStatusTimeoutFull);
       for (int j = 0; ok && j < n_blocks; ++j) {
         const int s = j & 1;                 // K stage
@@ -260,11 +267,12 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
             !mbar_wait(s_free(sb), uint32_t(j / Cfg::kSBufs - 1) & 1u, abort_flag, p.status, kStatusTimeoutTmemEmpty)) break;
         tc_fence_after();
         const uint64_t kd = s ? k_desc1 : k_desc0;
-        const uint32_t d_s = tmem_base + Cfg::kColS + sb * 128;
+        const uint32_t d_s = tmem_base + Cfg::kColS + sb * BKV;
 #pragma unroll
         for (int k = 0; k < D / 16; ++k) {
-          const uint64_t off = uint64_t(((k / 4) * (128 * 128) + (k % 4) * 32) >> 4);   // 16-byte units
-          umma_f16_ss(d_s, q_desc + off, kd + off, idesc_s, k > 0 ? 1u : 0u);
+          const uint64_t q_off = uint64_t(((k / 4) * (kFaBlockQ * 128) + (k % 4) * 32) >> 4);   // 16-byte units
+          const uint64_t k_off = uint64_t(((k / 4) * (BKV * 128) + (k % 4) * 32) >> 4);
+          umma_f16_ss(d_s, q_desc + q_off, kd + k_off, idesc_s, k > 0 ? 1u : 0u);
         }
         umma_commit(k_empty(s));
         umma_commit(s_full(sb));
@@ -273,11 +281,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   } else if (warp == 1) {
     // ---------------------------------------------------------------- PV MMA issuer (O_g += P V)
     if (lane == 0 && n_blocks > 0) {
-      constexpr uint32_t idesc_o = make_idesc_f16(kFaBlockQ, D, 1, 0, 1);
+      constexpr uint32_t idesc_o = make_idesc_f16(kFaBlockQ, DV, 1, 0, 1);
       uint64_t v_desc[2], p_desc[2];
 #pragma unroll
       for (int st = 0; st < 2; ++st) {
-        v_desc[st] = make_smem_desc_sw128(sbase + Cfg::kOffV + st * Cfg::kKVBytes, kFaBlockKV * 128, 1024);
+        v_desc[st] = make_smem_desc_sw128(sbase + Cfg::kOffV + st * Cfg::kVBytes, BKV * 128, 1024);
         p_desc[st] = make_smem_desc_sw128(sbase + Cfg::kOffP + st * Cfg::kPBytes, 16, 1024);
       }
       const bool trm = p.trace != nullptr && blockIdx.z == 0 && h == 0 && b == 0;
@@ -294,9 +302,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         tc_fence_after();
         const uint64_t pd = s ? p_desc[1] : p_desc[0];
         const uint64_t vd = s ? v_desc[1] : v_desc[0];
-        const uint32_t d_o = tmem_base + Cfg::kColO + s * D;
+        const uint32_t d_o = tmem_base + Cfg::kColO + s * DV;
 #pragma unroll
-        for (int k = 0; k < kFaBlockKV / 16; ++k) {
+        for (int k = 0; k < BKV / 16; ++k) {
           const uint64_t a_off = uint64_t(((k / 4) * (128 * 128) + (k % 4) * 32) >> 4);
           const uint64_t b_off = uint64_t((k * (16 * 128)) >> 4);
           umma_f16_ss(d_o, pd + a_off, vd + b_off, idesc_o, (j > 1 || k > 0) ? 1u : 0u);
@@ -319,7 +327,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const int row = quarter * 32 + lane;
     const int q_idx = q0 + row;
     const uint32_t lane_base = uint32_t(quarter * 32) << 16;
-    const uint32_t o_mine = tmem_base + lane_base + Cfg::kColO + grp * D;
+    const uint32_t o_mine = tmem_base + lane_base + Cfg::kColO + grp * DV;
     float m_used = 0.f, l = 0.f;
     bool seen = false;   // this row has met a visible key (with a window, whole blocks may lie before it)
     bool ok = true;
@@ -342,12 +350,12 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       int limit = p.Tk - 1 - kv0b;
       if (p.causal) limit = min(limit, q_base + row - kbase);
       const int lower = p.window > 0 ? q_base + row - kbase - p.window + 1 : 0;   // first visible column
-      const uint32_t s_mine = tmem_base + lane_base + Cfg::kColS + sb * 128;
+      const uint32_t s_mine = tmem_base + lane_base + Cfg::kColS + sb * BKV;
       // pass 1: row maximum (the scores are read from tensor memory twice, 64 columns at a time, instead of
       // holding all 128 in registers)
       float mx = -INFINITY;
 #pragma unroll 1
-      for (int hh = 0; hh < 2; ++hh) {
+      for (int hh = 0; hh < BKV / 64; ++hh) {
         uint32_t r[2][32];
         tmem_ld_32x32(s_mine + hh * 64, r[0]);
         tmem_ld_32x32(s_mine + hh * 64 + 32, r[1]);
@@ -382,7 +390,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           tc_fence_after();
           const float alpha = need ? ex2_approx_f(m_used - m_new) : 1.f;
 #pragma unroll
-          for (int c = 0; c < D / 16; ++c) {
+          for (int c = 0; c < DV / 16; ++c) {
             uint32_t o[16];
             tmem_ld_32x16(o_mine + c * 16, o);
             tmem_ld_wait();
@@ -404,7 +412,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       float sum = 0.f;
       uint8_t* prow = smem + Cfg::kOffP + grp * Cfg::kPBytes + (row >> 3) * 1024 + (row & 7) * 128;
 #pragma unroll 1
-      for (int hh = 0; hh < 2; ++hh) {
+      for (int hh = 0; hh < BKV / 64; ++hh) {
         uint32_t r[2][32];
         tmem_ld_32x32(s_mine + hh * 64, r[0]);
         tmem_ld_32x32(s_mine + hh * 64 + 32, r[1]);
@@ -477,11 +485,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       const float inv_l = (l_all > 0.f) ? 1.f / l_all : 0.f;
       const float w_mine = a_mine * inv_l, w_other = a_other * inv_l;
       if (n_blocks > 0) tc_fence_after();
-      __nv_bfloat16* orow = p.O + (long long)b * p.so_b + (long long)q_idx * p.so_t + (long long)h * D;
-      const uint32_t o_other = tmem_base + lane_base + Cfg::kColO + (grp ^ 1) * D;
-      // this warp writes output columns [grp * D / 2, (grp + 1) * D / 2) of its 32 rows
+      __nv_bfloat16* orow = p.O + (long long)b * p.so_b + (long long)q_idx * p.so_t + (long long)h * DV;
+      const uint32_t o_other = tmem_base + lane_base + Cfg::kColO + (grp ^ 1) * DV;
+      // this warp writes output columns [grp * DV / 2, (grp + 1) * DV / 2) of its 32 rows
 #pragma unroll 1
-      for (int c = grp * (D / 32); c < (grp + 1) * (D / 32); ++c) {
+      for (int c = grp * (DV / 32); c < (grp + 1) * (DV / 32); ++c) {
         uint32_t o[16], o2[16];
         if (mine_used) tmem_ld_32x16(o_mine + c * 16, o);
         if (other_used) tmem_ld_32x16(o_other + c * 16, o2);
@@ -525,11 +533,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 
 static long long* g_fwd_trace = nullptr;
 
-template <int D>
+template <int D, int DV = D, int BKV = kFaBlockKV, bool SHARED = false>
 static int launch_flash_fwd(const CUtensorMap& tq, const KvMaps& maps, const FlashFwdParams& p, cudaStream_t st) {
-  using Cfg = FaFwdCfg<D>;
+  using Cfg = FaFwdCfg<D, DV, BKV>;
   static bool configured = false;
-  auto kern = flash_fwd_kernel<D>;
+  auto kern = flash_fwd_kernel<D, DV, BKV, SHARED>;
   if (!configured) {
     LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
     configured = true;
@@ -577,6 +585,43 @@ static int flash_fwd_common(const void* q, const void* const* k_ptrs, const void
   return D == 64 ? launch_flash_fwd<64>(tq, maps, p, st) : launch_flash_fwd<128>(tq, maps, p, st);
 }
 
+// One sequence whose keys are [the head's own columns | 64 columns shared by all heads].
+static int flash_fwd_shared(const void* q, const void* k, const void* k_shared, const void* v, void* o, float* lse, int Tq, int Tk, int H,
+                            int D, int DV, long long sq_t, long long sk_t, long long ss_t, long long sv_t, float scale, int window,
+                            cudaStream_t st) {
+  const bool wide = D == 192 && DV == 128, mid = D == 128 && (DV == 64 || DV == 128);
+  if ((!wide && !mid) || H < 1 || Tk < Tq || window < 0) return -int(kStatusBadArgument);
+  if (Tq == 0) return 0;
+  const int block_kv = wide ? 64 : kFaBlockKV, dk = D - 64;
+  // one batch entry: its stride is never used, but has to be a valid one
+  auto map = [&](CUtensorMap* m, const void* base, int cols, int heads, int rows, long long pitch, int box_rows) {
+    return encode_tmap_4d(m, base, 2, cols, heads, rows, 1, (uint64_t)cols * 2, (uint64_t)pitch * 2, (uint64_t)pitch * rows * 2, 64, 1,
+                          box_rows, 1, 1);
+  };
+  CUtensorMap tq;
+  KvMaps maps;
+  int r = map(&tq, q, D, H, Tq, sq_t, kFaBlockQ);
+  if (r) return 1000 + r;
+  for (int i = 0; i < kFaMaxRanks; ++i) {
+    r = i == 0 ? map(&maps.k[i], k, dk, H, Tk, sk_t, block_kv) : map(&maps.k[i], k_shared, 64, 1, Tk, ss_t, block_kv);
+    if (r) return 2000 + r;
+    r = map(&maps.v[i], v, DV, H, Tk, sv_t, block_kv);
+    if (r) return 3000 + r;
+  }
+  FlashFwdParams p{};
+  p.O = static_cast<__nv_bfloat16*>(o);
+  p.lse = lse;
+  p.B = 1; p.Tq = Tq; p.Tk = Tk; p.Hq = H; p.Hkv = H;
+  p.so_b = (long long)Tq * H * DV; p.so_t = (long long)H * DV;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.causal = 1;
+  p.cp_world = 1;
+  p.window = window;
+  p.status = device_status_word();
+  if (wide) return launch_flash_fwd<192, 128, 64, true>(tq, maps, p, st);
+  return DV == 64 ? launch_flash_fwd<128, 64, kFaBlockKV, true>(tq, maps, p, st) : launch_flash_fwd<128, 128, kFaBlockKV, true>(tq, maps, p, st);
+}
+
 }  // namespace lt
 
 extern "C" {
@@ -605,6 +650,15 @@ int lt_flash_fwd_window(const void* q, const void* k, const void* v, void* o, fl
   const void* vs[1] = {v};
   return lt::flash_fwd_common(q, ks, vs, o, lse, B, Tq, Tk, Hq, Hkv, D, sq_b, sq_t, sk_b, sk_t, sv_b, sv_t, so_b, so_t, scale,
                               1, 1, 0, 0, window, stream);
+}
+
+// Causal attention of one sequence with keys in two parts: q [Tq, H, D], k [Tk, H, D - 64], k_shared [Tk, 64] (the last 64 columns of
+// every head's keys), v [Tk, H, DV], o [Tq, H, DV] packed; heads are packed, rows at the given pitches (multiples of 8 elements).
+// The last query stands on the last key; window as above, 0: none.  (D, DV) is (128, 64), (128, 128) or (192, 128).
+int lt_flash_fwd_shared(const void* q, const void* k, const void* k_shared, const void* v, void* o, float* lse, int Tq, int Tk, int H,
+                        int D, int DV, long long sq_t, long long sk_t, long long ss_t, long long sv_t, float scale, int window,
+                        void* stream) {
+  return lt::flash_fwd_shared(q, k, k_shared, v, o, lse, Tq, Tk, H, D, DV, sq_t, sk_t, ss_t, sv_t, scale, window, static_cast<cudaStream_t>(stream));
 }
 
 // Context-parallel forward: k_ptrs[r] / v_ptrs[r] are rank r's KV shards [B, Tk, Hkv, D] (peer-mapped pointers, all with

@@ -1,6 +1,7 @@
 // GEMM on the CUDA cores for what the tensor-core kernels do not take: true fp32 operands (no reduced-precision mode) and
 // bf16 operands whose pitch or inner extent TMA cannot describe.  Optionally a batch of equal products at fixed element
-// offsets (a block-diagonal matrix is one).  Also the narrow projection with fp32 results (gates of a recurrence).
+// offsets (a block-diagonal matrix is one), or rows grouped by expert (a mixture of experts).  Also the narrow projection with
+// fp32 results (gates of a recurrence, a router).
 #include "lt_cuda.h"
 #include "common/host.h"
 #include "common/scalar.cuh"
@@ -9,16 +10,36 @@ namespace lt {
 
 constexpr int kStTile = 64, kStK = 16;
 
+// Rows in blocks of kStTile, each with the matrix of one expert (see lt_gemm_simt_grouped).
+struct StGroups {
+  const int* group;
+  const int* rows;
+  const int* live;
+  const int* src;
+};
+
 // C[M, N] = alpha * A[M, K] @ B[N, K]^T; 256 threads, 4 x 4 results each, fp32 accumulation in blocks of kStK (a sum of short
 // sums: the rounding error grows with the number of blocks, not with K).
-template <typename T, typename TO>
+template <typename T, typename TO, bool GROUPED>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, TO* __restrict__ C, int M, int N, int K, long long lda,
-                 long long ldb, long long ldc, long long sa, long long sb, long long sc, float alpha) {
+                 long long ldb, long long ldc, long long sa, long long sb, long long sc, float alpha, const StGroups gr) {
   __shared__ float As[kStK][kStTile + 4], Bs[kStK][kStTile + 4];
-  A += blockIdx.z * sa;
-  B += blockIdx.z * sb;
-  C += blockIdx.z * sc;
+  __shared__ int row_of[kStTile];
+  if constexpr (GROUPED) {
+    if (int(blockIdx.y) >= *gr.live) return;
+    M = blockIdx.y * kStTile + gr.rows[blockIdx.y];
+    B += gr.group[blockIdx.y] * sb;
+    if (threadIdx.x < kStTile) {
+      const int m = blockIdx.y * kStTile + threadIdx.x;
+      row_of[threadIdx.x] = !gr.src ? m : m < M ? gr.src[m] : 0;
+    }
+    __syncthreads();
+  } else {
+    A += blockIdx.z * sa;
+    B += blockIdx.z * sb;
+    C += blockIdx.z * sc;
+  }
   const int m0 = blockIdx.y * kStTile, n0 = blockIdx.x * kStTile;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
@@ -27,7 +48,7 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, TO* __restric
     for (int i = 0; i < 4; ++i) {
       const int e = threadIdx.x + i * 256;
       const int r = e >> 4, k = k0 + (e & 15);
-      As[e & 15][r] = (m0 + r < M && k < K) ? ldf(A + (m0 + r) * lda + k) : 0.f;
+      As[e & 15][r] = (m0 + r < M && k < K) ? ldf(A + (GROUPED ? row_of[r] : m0 + r) * lda + k) : 0.f;
       Bs[e & 15][r] = (n0 + r < N && k < K) ? ldf(B + (n0 + r) * ldb + k) : 0.f;
     }
     __syncthreads();
@@ -113,13 +134,32 @@ int lt_gemm_simt(int in_fp32, int out_fp32, const void* A, const void* B, void* 
   dim3 grid((N + kStTile - 1) / kStTile, mb, batch);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   using bf = __nv_bfloat16;
-#define LT_ST(TI, TO) gemm_simt_kernel<TI, TO><<<grid, 256, 0, st>>>(static_cast<const TI*>(A), static_cast<const TI*>(B), \
-                                                                     static_cast<TO*>(C), M, N, K, lda, ldb, ldc, sa, sb, sc, alpha)
+#define LT_ST(TI, TO) gemm_simt_kernel<TI, TO, false><<<grid, 256, 0, st>>>( \
+      static_cast<const TI*>(A), static_cast<const TI*>(B), static_cast<TO*>(C), M, N, K, lda, ldb, ldc, sa, sb, sc, alpha, StGroups{})
   if (in_fp32 && out_fp32) LT_ST(float, float);
   else if (!in_fp32 && out_fp32) LT_ST(bf, float);
   else if (!in_fp32) LT_ST(bf, bf);
   else return -4;
 #undef LT_ST
+  LT_LAUNCH_CHECK();
+  return 0;
+}
+
+// Rows grouped by expert in blocks of 64: block b (of *live, at most max_blocks) takes rows src[64 b ..] of A (src nullptr: the same
+// rows), group_rows[b] of them, times B[group[b]] ([experts, N, K]), into rows 64 b .. of C.  A, B and C of one type.
+int lt_gemm_simt_grouped(int fp32, const void* A, long long lda, const void* B, void* C, const int* group, const int* group_rows,
+                         const int* live, const int* src, int max_blocks, int N, int K, void* stream) {
+  using namespace lt;
+  if (max_blocks < 1 || max_blocks > 65535 || N < 1 || K < 1) return -4;
+  dim3 grid((N + kStTile - 1) / kStTile, max_blocks);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const StGroups gr{group, group_rows, live, src};
+  using bf = __nv_bfloat16;
+#define LT_SG(T) gemm_simt_kernel<T, T, true><<<grid, 256, 0, st>>>(static_cast<const T*>(A), static_cast<const T*>(B), static_cast<T*>(C), \
+                                                                    0, N, K, lda, K, N, 0, (long long)N * K, 0, 1.f, gr)
+  if (fp32) LT_SG(float);
+  else LT_SG(bf);
+#undef LT_SG
   LT_LAUNCH_CHECK();
   return 0;
 }

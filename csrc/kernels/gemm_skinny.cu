@@ -10,11 +10,18 @@
 // The eight warps' partial sums are folded through shared memory; when several CTAs share a column group (narrow
 // outputs: more CTAs than column groups are needed to fill the GPU) each writes its partial to a workspace and the CTA
 // that arrives last at the group's counter adds them in a fixed order, so the result does not depend on arrival order
-// and nothing ever waits.  The reference runs every Linear through cublasSgemm whatever the row count
+// and nothing ever waits.
+//
+// Three variants share the loop: a batch of equal products at fixed offsets (one per attention head), rows grouped by expert
+// (a mixture of experts in a decode step: blocks of 16, 32 or 64 rows, each block with the matrix of its expert, its
+// rows picked out of the tokens by a table), and a gated epilogue: w holds gate rows, then up rows, a CTA owns 16 of
+// each, and y = act(gate) * up leaves the kernel, so that the wide intermediate is never stored.
+// The reference runs every Linear through cublasSgemm whatever the row count
 // (src/ops/linear.cpp:176-192).
 #include "lt_cuda.h"
 #include "common/host.h"
 #include "common/ptx.cuh"
+#include "common/scalar.cuh"
 
 #include <atomic>
 #include <map>
@@ -36,21 +43,72 @@ __device__ __forceinline__ void mma_bf16_16816(float (&d)[4], uint32_t a0, uint3
       : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-// MT = number of 16-row blocks of x (rows past M read as zero).  Grid: (column groups, K splits).
-template <int MT>
-__global__ void __launch_bounds__(kSkWarps * 32, 1)
-gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __nv_bfloat16* __restrict__ w, long long ldw,
-                   __nv_bfloat16* __restrict__ y, long long ldy, const __nv_bfloat16* __restrict__ residual, long long ldr,
-                   int M, int N, int K, int chunks_per_cta, float* __restrict__ ws, unsigned* __restrict__ counters) {
+struct SkinnyParams {
+  const __nv_bfloat16* x;
+  long long ldx;
+  const __nv_bfloat16* w;
+  long long ldw;
+  __nv_bfloat16* y;
+  long long ldy;
+  const __nv_bfloat16* residual;
+  long long ldr;
+  int M, N, K, chunks_per_cta;   // gated: N counts results, w has 2 N rows
+  float* ws;
+  unsigned* counters;
+  int act;                       // gated: 1 GELU (tanh form), 2 SiLU
+  long long sx, sw, sy;          // batch: element offsets of the next product; grouped: sw of the next expert's matrix
+  const int* group;              // grouped: expert of every block of 16 MT rows
+  const int* group_rows;         // rows of the block that exist
+  const int* live;               // number of blocks
+  const int* src;                // row of x for every row of y; nullptr: the same row
+};
+
+enum { kSkPlain = 0, kSkBatch = 1, kSkGrouped = 2 };
+
+// MT = number of 16-row blocks of x (rows past M read as zero).  Grid: (column groups, K splits, products or row blocks).
+template <int MT, int MODE, bool GLU>
+__global__ void __launch_bounds__(kSkWarps * 32, (MODE != kSkPlain || GLU) && MT == 1 ? 2 : 1)
+gemm_skinny_kernel(const SkinnyParams p) {
   extern __shared__ float red[];   // [4 slots][MT * 16 registers][32 lanes]
   constexpr int R = MT * 16;
   constexpr int U = MT <= 2 ? 4 : 2;   // chunks whose weight loads are in flight together
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, q = lane & 3;
-  const int n0 = blockIdx.x * kSkCols;
-  const int nchunks = K >> 5;
-  const int c_begin = blockIdx.y * chunks_per_cta;
-  const int c_end = min(nchunks, c_begin + chunks_per_cta);
+  const int n0 = blockIdx.x * (GLU ? kSkCols / 2 : kSkCols);
+  const int nchunks = p.K >> 5;
+  const int c_begin = blockIdx.y * p.chunks_per_cta;
+  const int c_end = min(nchunks, c_begin + p.chunks_per_cta);
+  const int N = p.N;
+  int M = p.M;
+  const __nv_bfloat16* x = p.x;
+  const __nv_bfloat16* w = p.w;
+  __nv_bfloat16* y = p.y;
+  if constexpr (MODE == kSkBatch) {
+    x += blockIdx.z * p.sx;
+    w += blockIdx.z * p.sw;
+    y += blockIdx.z * p.sy;
+  }
+  if constexpr (MODE == kSkGrouped) {
+    if (int(blockIdx.z) >= *p.live) return;
+    M = p.group_rows[blockIdx.z];
+    w += p.group[blockIdx.z] * p.sw;
+    y += (long long)blockIdx.z * R * p.ldy;
+  }
+  // the rows of x this lane reads
+  const __nv_bfloat16* xrow[MT][2];
+  if constexpr (MODE == kSkGrouped) {
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int r = m * 16 + g + h * 8;
+        long long at = (long long)blockIdx.z * R + r;
+        if (p.src) at = r < M ? p.src[at] : 0;
+        xrow[m][h] = x + at * p.ldx + q * 8;
+      }
+  }
+  const __nv_bfloat16* xbase = x + q * 8;
+  const long long ldx = p.ldx;
 
   float acc[MT][4][4];
 #pragma unroll
@@ -64,11 +122,10 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __n
   bool wok[4];
 #pragma unroll
   for (int f = 0; f < 4; ++f) {
-    const int n = n0 + f * 8 + g;
+    const int n = n0 + (GLU ? f & 1 : f) * 8 + g;
     wok[f] = n < N;
-    wrow[f] = w + (long long)(wok[f] ? n : 0) * ldw + q * 8;
+    wrow[f] = w + (long long)(wok[f] ? n + (GLU && f >= 2 ? N : 0) : 0) * p.ldw + q * 8;
   }
-  const __nv_bfloat16* xbase = x + q * 8;
 
   for (int c = c_begin + warp; c < c_end; c += kSkWarps * U) {
     uint4 wv[U][4];
@@ -87,8 +144,11 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __n
       for (int m = 0; m < MT; ++m) {
         const int r0 = m * 16 + g, r1 = r0 + 8;
         const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-        const uint4 xlo = r0 < M ? __ldg(reinterpret_cast<const uint4*>(xbase + (long long)r0 * ldx + cc * 32)) : zero;
-        const uint4 xhi = r1 < M ? __ldg(reinterpret_cast<const uint4*>(xbase + (long long)r1 * ldx + cc * 32)) : zero;
+        const __nv_bfloat16 *x0, *x1;
+        if constexpr (MODE == kSkGrouped) { x0 = xrow[m][0]; x1 = xrow[m][1]; }
+        else { x0 = xbase + (long long)r0 * ldx; x1 = xbase + (long long)r1 * ldx; }
+        const uint4 xlo = r0 < M ? __ldg(reinterpret_cast<const uint4*>(x0 + cc * 32)) : zero;
+        const uint4 xhi = r1 < M ? __ldg(reinterpret_cast<const uint4*>(x1 + cc * 32)) : zero;
 #pragma unroll
         for (int f = 0; f < 4; ++f) {
           // physical k = q * 8 + j * 4 + {0, 1} plays logical k = q * 2 + {0, 1}, physical + 2 plays logical + 8, for A and B alike
@@ -127,7 +187,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __n
 
   const int splits = gridDim.y;
   if (splits > 1) {
-    float* mine = ws + ((size_t)blockIdx.y * gridDim.x + blockIdx.x) * (R * 32) + lane;
+    float* mine = p.ws + ((size_t)blockIdx.y * gridDim.x + blockIdx.x) * (R * 32) + lane;
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -137,7 +197,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __n
     __threadfence();
     __syncwarp();
     unsigned prev = 0;
-    if (lane == 0) prev = atomicAdd(counters + blockIdx.x, 1u);
+    if (lane == 0) prev = atomicAdd(p.counters + blockIdx.x, 1u);
     prev = __shfl_sync(0xffffffffu, prev, 0);
     if (prev != unsigned(splits - 1)) return;   // not the last CTA of this column group
     __threadfence();
@@ -148,7 +208,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __n
 #pragma unroll
         for (int r = 0; r < 4; ++r) acc[m][f][r] = 0.f;
     for (int s = 0; s < splits; ++s) {   // every part from the workspace, in index order: the sum is the same whoever is last
-      const float* part = ws + ((size_t)s * gridDim.x + blockIdx.x) * (R * 32) + lane;
+      const float* part = p.ws + ((size_t)s * gridDim.x + blockIdx.x) * (R * 32) + lane;
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -156,13 +216,13 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __n
 #pragma unroll
           for (int r = 0; r < 4; ++r) acc[m][f][r] += __ldcg(part + ((m * 4 + f) * 4 + r) * 32);
     }
-    if (lane == 0) counters[blockIdx.x] = 0u;   // ready for the next launch on this stream
+    if (lane == 0) p.counters[blockIdx.x] = 0u;   // ready for the next launch on this stream
   }
 
 #pragma unroll
   for (int m = 0; m < MT; ++m) {
 #pragma unroll
-    for (int f = 0; f < 4; ++f) {
+    for (int f = 0; f < (GLU ? 2 : 4); ++f) {
       const int col = n0 + f * 8 + q * 2;
       if (col >= N) continue;
 #pragma unroll
@@ -170,12 +230,16 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __n
         const int row = m * 16 + g + h * 8;
         if (row >= M) continue;
         float v0 = acc[m][f][h * 2], v1 = acc[m][f][h * 2 + 1];
-        if (residual) {
-          const float2 rv = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(residual + (long long)row * ldr + col));
+        if constexpr (GLU) {
+          const float u0 = acc[m][f + 2][h * 2], u1 = acc[m][f + 2][h * 2 + 1];
+          v0 = (p.act == 1 ? gelu_tanh_f(v0) : v0 * sigmoid_f(v0)) * u0;
+          v1 = (p.act == 1 ? gelu_tanh_f(v1) : v1 * sigmoid_f(v1)) * u1;
+        } else if (p.residual) {
+          const float2 rv = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p.residual + (long long)row * p.ldr + col));
           v0 += rv.x;
           v1 += rv.y;
         }
-        *reinterpret_cast<uint32_t*>(y + (long long)row * ldy + col) = pack_bf16x2(v0, v1);
+        *reinterpret_cast<uint32_t*>(y + (long long)row * p.ldy + col) = pack_bf16x2(v0, v1);
       }
     }
   }
@@ -226,20 +290,20 @@ static bool get_skinny_ws(cudaStream_t st, SkinnyWs* out) {
   return true;
 }
 
-template <int MT>
-static int launch_skinny(const __nv_bfloat16* X, long long ldx, const __nv_bfloat16* W, long long ldw, __nv_bfloat16* Y, long long ldy,
-                         const __nv_bfloat16* R, long long ldr, int M, int N, int K, cudaStream_t st) {
+template <int MT, int MODE, bool GLU>
+static int launch_skinny(SkinnyParams p, int z, cudaStream_t st) {
   static bool configured = false;
   constexpr int smem = 4 * MT * 16 * 32 * 4;
-  auto kern = gemm_skinny_kernel<MT>;
+  auto kern = gemm_skinny_kernel<MT, MODE, GLU>;
   if (!configured) {
     LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     configured = true;
   }
   const int sms = sm_count();
-  const int groups = (N + kSkCols - 1) / kSkCols;
-  const int nchunks = K / 32;
-  int splits = (g_sk_target.load() * sms + groups - 1) / groups;
+  const int cols = GLU ? kSkCols / 2 : kSkCols;
+  const int groups = (p.N + cols - 1) / cols;
+  const int nchunks = p.K / 32;
+  int splits = MODE == kSkPlain ? (g_sk_target.load() * sms + groups - 1) / groups : 1;
   const int mc = g_sk_min_chunks.load();
   const int max_splits = nchunks / (mc * kSkWarps) > 1 ? nchunks / (mc * kSkWarps) : 1;   // at least `mc` chunks per warp
   if (splits > max_splits) splits = max_splits;
@@ -250,10 +314,27 @@ static int launch_skinny(const __nv_bfloat16* X, long long ldx, const __nv_bfloa
   }
   int per = (nchunks + splits - 1) / splits;
   splits = (nchunks + per - 1) / per;
-  dim3 grid(groups, splits);
-  kern<<<grid, kSkWarps * 32, smem, st>>>(X, ldx, W, ldw, Y, ldy, R, ldr, M, N, K, per, wsp.ws, wsp.counters);
+  p.chunks_per_cta = per;
+  p.ws = wsp.ws;
+  p.counters = wsp.counters;
+  kern<<<dim3(groups, splits, z), kSkWarps * 32, smem, st>>>(p);
   LT_LAUNCH_CHECK();
   return 0;
+}
+
+template <int MODE, bool GLU>
+static int skinny_by_rows(const SkinnyParams& p, int rows, int z, cudaStream_t st) {
+  if (rows <= 16) return launch_skinny<1, MODE, GLU>(p, z, st);
+  if (rows <= 32) return launch_skinny<2, MODE, GLU>(p, z, st);
+  if (rows <= 64) return launch_skinny<4, MODE, GLU>(p, z, st);
+  if constexpr (MODE == kSkGrouped) return -int(kStatusBadArgument);
+  else return launch_skinny<8, MODE, GLU>(p, z, st);
+}
+
+static bool skinny_ok(const SkinnyParams& p) {
+  return p.N > 0 && p.K > 0 && !(p.K & 31) && !(p.N & 7) && !(p.ldx & 7) && !(p.ldw & 7) && !(p.ldy & 1) && !(p.ldr & 1) &&
+         !(p.sx & 7) && !(p.sw & 7) && !(p.sy & 1) && !(reinterpret_cast<uintptr_t>(p.x) & 15) && !(reinterpret_cast<uintptr_t>(p.w) & 15) &&
+         !(reinterpret_cast<uintptr_t>(p.y) & 3) && !(reinterpret_cast<uintptr_t>(p.residual) & 3);
 }
 
 }  // namespace lt
@@ -273,19 +354,58 @@ int lt_gemm_skinny_set_target(int ctas_per_sm, int min_chunks_per_warp) {
 int lt_gemm_skinny_bf16(const void* x, long long ldx, const void* w, long long ldw, void* y, long long ldy, const void* residual,
                         long long ldr, int M, int N, int K, void* stream) {
   using namespace lt;
-  if (M < 1 || M > 128 || N <= 0 || K <= 0 || (K & 31) || (N & 7) || (ldx & 7) || (ldw & 7) || (ldy & 1) || (ldr & 1) ||
-      (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) || (reinterpret_cast<uintptr_t>(y) & 3) ||
-      (reinterpret_cast<uintptr_t>(residual) & 3))
+  SkinnyParams p{};
+  p.x = static_cast<const __nv_bfloat16*>(x); p.ldx = ldx;
+  p.w = static_cast<const __nv_bfloat16*>(w); p.ldw = ldw;
+  p.y = static_cast<__nv_bfloat16*>(y); p.ldy = ldy;
+  p.residual = static_cast<const __nv_bfloat16*>(residual); p.ldr = ldr;
+  p.M = M; p.N = N; p.K = K;
+  if (M < 1 || M > 128 || !skinny_ok(p)) return -int(kStatusBadArgument);
+  return skinny_by_rows<kSkPlain, false>(p, M, 1, static_cast<cudaStream_t>(stream));
+}
+
+// y[M, N] = act(x @ gate^T) * (x @ up^T), w [2 N, K] = gate rows, then up rows; act 1: GELU (tanh form), 2: SiLU.  Otherwise as above.
+int lt_gemm_skinny_glu(const void* x, long long ldx, const void* w, void* y, int M, int N, int K, int act, void* stream) {
+  using namespace lt;
+  SkinnyParams p{};
+  p.x = static_cast<const __nv_bfloat16*>(x); p.ldx = ldx;
+  p.w = static_cast<const __nv_bfloat16*>(w); p.ldw = K;
+  p.y = static_cast<__nv_bfloat16*>(y); p.ldy = N;
+  p.M = M; p.N = N; p.K = K; p.act = act;
+  if (M < 1 || M > 128 || act < 1 || act > 2 || !skinny_ok(p)) return -int(kStatusBadArgument);
+  return skinny_by_rows<kSkPlain, true>(p, M, 1, static_cast<cudaStream_t>(stream));
+}
+
+// A batch of products y_b = x_b @ w_b^T: x_b at offset b * sx, w_b [N, K] one after another, y_b at offset b * sy.
+int lt_gemm_skinny_batch(const void* x, long long ldx, long long sx, const void* w, void* y, long long ldy, long long sy, int batch,
+                         int M, int N, int K, void* stream) {
+  using namespace lt;
+  SkinnyParams p{};
+  p.x = static_cast<const __nv_bfloat16*>(x); p.ldx = ldx; p.sx = sx;
+  p.w = static_cast<const __nv_bfloat16*>(w); p.ldw = K; p.sw = (long long)N * K;
+  p.y = static_cast<__nv_bfloat16*>(y); p.ldy = ldy; p.sy = sy;
+  p.M = M; p.N = N; p.K = K;
+  if (M < 1 || M > 128 || batch < 1 || batch > 65535 || !skinny_ok(p)) return -int(kStatusBadArgument);
+  return skinny_by_rows<kSkBatch, false>(p, M, batch, static_cast<cudaStream_t>(stream));
+}
+
+// Rows grouped by expert in blocks of block_rows (16, 32 or 64): block b (of *live, at most max_blocks) takes rows of x
+// src[b block_rows ..] (src nullptr: the same rows of x), group_rows[b] of them, times the matrix of expert group[b], into
+// rows b block_rows .. of y.  act 0: w [experts, N, K]; else gated as in lt_gemm_skinny_glu, w [experts, 2 N, K].
+int lt_gemm_skinny_grouped(const void* x, long long ldx, const void* w, void* y, const int* group, const int* group_rows,
+                           const int* live, const int* src, int max_blocks, int block_rows, int N, int K, int act, void* stream) {
+  using namespace lt;
+  SkinnyParams p{};
+  p.x = static_cast<const __nv_bfloat16*>(x); p.ldx = ldx;
+  p.w = static_cast<const __nv_bfloat16*>(w); p.ldw = K; p.sw = (long long)(act ? 2 * N : N) * K;
+  p.y = static_cast<__nv_bfloat16*>(y); p.ldy = N;
+  p.N = N; p.K = K; p.act = act;
+  p.group = group; p.group_rows = group_rows; p.live = live; p.src = src;
+  if (max_blocks < 1 || max_blocks > 65535 || act < 0 || act > 2 || (block_rows != 16 && block_rows != 32 && block_rows != 64) ||
+      !skinny_ok(p))
     return -int(kStatusBadArgument);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  auto X = static_cast<const __nv_bfloat16*>(x);
-  auto W = static_cast<const __nv_bfloat16*>(w);
-  auto Y = static_cast<__nv_bfloat16*>(y);
-  auto R = static_cast<const __nv_bfloat16*>(residual);
-  if (M <= 16) return launch_skinny<1>(X, ldx, W, ldw, Y, ldy, R, ldr, M, N, K, st);
-  if (M <= 32) return launch_skinny<2>(X, ldx, W, ldw, Y, ldy, R, ldr, M, N, K, st);
-  if (M <= 64) return launch_skinny<4>(X, ldx, W, ldw, Y, ldy, R, ldr, M, N, K, st);
-  return launch_skinny<8>(X, ldx, W, ldw, Y, ldy, R, ldr, M, N, K, st);
+  return act ? skinny_by_rows<kSkGrouped, true>(p, block_rows, max_blocks, st) : skinny_by_rows<kSkGrouped, false>(p, block_rows, max_blocks, st);
 }
 
 }  // extern "C"

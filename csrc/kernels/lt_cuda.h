@@ -50,6 +50,9 @@ int lt_flash_fwd_cp(const void* q, const void* const* k_ptrs, const void* const*
 int lt_flash_fwd_window(const void* q, const void* k, const void* v, void* o, float* lse, int B, int Tq, int Tk, int Hq,
                         int Hkv, int D, long long sq_b, long long sq_t, long long sk_b, long long sk_t, long long sv_b,
                         long long sv_t, long long so_b, long long so_t, float scale, int window, void* stream);
+int lt_flash_fwd_shared(const void* q, const void* k, const void* k_shared, const void* v, void* o, float* lse, int Tq, int Tk, int H,
+                        int D, int DV, long long sq_t, long long sk_t, long long ss_t, long long sv_t, float scale, int window,
+                        void* stream);
 
 // ---- fsdp_fused.cu: ZeRO-3 fused paths: all-gather -> GEMM, reduce-scatter -> AdamW, shard gathers, flag barrier between ranks
 int lt_ag_gemm_bf16(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
@@ -85,6 +88,11 @@ int lt_quant_fp8_1x128(const void* x, long long ldx, void* q, long long ldq, voi
 int lt_gemm_skinny_set_target(int ctas_per_sm, int min_chunks_per_warp);
 int lt_gemm_skinny_bf16(const void* x, long long ldx, const void* w, long long ldw, void* y, long long ldy,
                         const void* residual, long long ldr, int M, int N, int K, void* stream);
+int lt_gemm_skinny_glu(const void* x, long long ldx, const void* w, void* y, int M, int N, int K, int act, void* stream);
+int lt_gemm_skinny_batch(const void* x, long long ldx, long long sx, const void* w, void* y, long long ldy, long long sy, int batch,
+                         int M, int N, int K, void* stream);
+int lt_gemm_skinny_grouped(const void* x, long long ldx, const void* w, void* y, const int* group, const int* group_rows,
+                           const int* live, const int* src, int max_blocks, int block_rows, int N, int K, int act, void* stream);
 
 // ---- gemm_sm100.cu: persistent tcgen05 GEMM: C = epilogue(alpha * op(A) op(B)); a_major / b_major 0 = K contiguous; act 1 = GELU;
 // pitches in elements; returns 0, a cudaError_t, or 1000 + CUresult of a failed tensor-map encoding
@@ -177,9 +185,25 @@ int lt_hyper_norm(int fp32, void* x, const int* tokens, const void* embed, const
                   const float* norm, float eps, void* h, long long ldh, const int* rows, int n_rows, int width, int streams,
                   int write_x, void* stream);
 
+// ---- residual_norm.cu, latent_attn.cu, moe_serve.cu: single residual with norms on both sides, latent attention, mixture of experts
+int lt_residual_norm(int fp32, float* x, const int* tokens, const void* embed, const void* y, long long ldy, const void* z,
+                     const int* z_slot, const float* z_weight, int top, const float* y_norm, float mult, const float* norm, float eps,
+                     void* h, const int* rows, int n_rows, int width, int write_x, void* stream);
+int lt_latent_rope(int fp32, void* proj, long long ld, int n, int H, int d, int r, int rot, int c_off, int rank, int c,
+                   const float* c_norm, float eps, const int* positions, const int* slots, const double* freq, float gain, void* q_out,
+                   int q_ld, int q_col, void* cache, void* lin, void* stream);
+int lt_latent_decode(const void* q, const void* cache, const int* tables, const int* ctx, float* part, float* stat, void* out, int S,
+                     int H, int c, int w, int block_size, int max_blocks, int splits, int window, float scale, void* stream);
+int lt_moe_plan(const float* logits, const float* correction, float* weight, int* slot, int* src, int* group, int* group_rows, int* live,
+                void* pairs, int* counts, const void* x, void* xs, int row_bytes, int N, int E, int top, int block_rows, void* stream);
+int lt_moe_grouped_gemm(const void* A, const void* W, void* C, const int* group, const int* live, int max_blocks, int experts, int N,
+                        int K, void* stream);
+
 // ---- gemm_simt.cu: CUDA-core GEMM (true fp32, odd shapes, batches) and narrow projections with fp32 results
 int lt_gemm_simt(int in_fp32, int out_fp32, const void* A, const void* B, void* C, int M, int N, int K, long long lda,
                  long long ldb, long long ldc, int batch, long long sa, long long sb, long long sc, float alpha, void* stream);
+int lt_gemm_simt_grouped(int fp32, const void* A, long long lda, const void* B, void* C, const int* group, const int* group_rows,
+                         const int* live, const int* src, int max_blocks, int N, int K, void* stream);
 int lt_rows_dot(int fp32, const void* x, long long ldx, const void* w, float* y, int R, int J, int K, void* stream);
 
 // ---- window_attn.cu: projection norm + rotary embedding + cache write, window gather, CUDA-core attention, head gates
@@ -234,6 +258,9 @@ int lt_rope(void* x, const float* cos_t, const float* sin_t, const int* pos, lon
             long long row_stride, int backward, void* stream);
 int lt_swiglu_fwd(const void* gu, void* h, long long M, int F, void* stream);
 int lt_clamped_glu(int fp32, const void* gu, void* h, long long M, int F, float limit, float slope, void* stream);
+int lt_act_glu(int fp32, const void* gu, void* h, long long M, int F, int act, const int* live, int block_rows, void* stream);
+int lt_token_gate(int fp32, const void* g, const int* tokens, const void* table, long long ldt, int off, int dim, int ld, void* out,
+                  int n, void* stream);
 int lt_swiglu_bwd(const void* gu, const void* dh, void* dgu, long long M, int F, void* stream);
 int lt_gelu_fwd(const void* x, void* y, long long n, void* stream);
 int lt_gelu_bwd(const void* x, const void* dy, void* dx, long long n, void* stream);

@@ -107,6 +107,47 @@ __global__ void clamped_glu8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_b
   }
 }
 
+// h = act(gate) * up; act 1: GELU (tanh form), 2: SiLU.  `live` (nullptr: all M rows) counts blocks of block_rows rows in use.
+// V: columns per thread (1, or 8 for bf16).
+template <typename T, int V>
+__global__ void act_glu_kernel(const T* __restrict__ gu, T* __restrict__ h, long long M, int F, int act, const int* __restrict__ live,
+                               int block_rows) {
+  if (live) M = min(M, (long long)*live * block_rows);
+  const int fv = F / V;
+  const long long total = M * fv;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / fv;
+    const int c = int(i - r * fv) * V;
+    float g[V], u[V];
+    if constexpr (V == 8) {
+      ldf8(gu + r * 2 * F + c, g);
+      ldf8(gu + r * 2 * F + F + c, u);
+    } else {
+      g[0] = ldf(gu + r * 2 * F + c);
+      u[0] = ldf(gu + r * 2 * F + F + c);
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) g[k] = (act == 1 ? gelu_tanh_f(g[k]) : g[k] * sigmoid_f(g[k])) * u[k];
+    if constexpr (V == 8) {
+      *reinterpret_cast<uint4*>(h + r * F + c) =
+          make_uint4(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]), pack_bf16x2(g[4], g[5]), pack_bf16x2(g[6], g[7]));
+    } else {
+      stf(h + r * F + c, g[0]);
+    }
+  }
+}
+
+// out[n, c] = gelu(g[n, c]) * table[tokens[n], off + c] for c < dim, zero up to ld: a token's own input, gated.
+template <typename T>
+__global__ void token_gate_kernel(const T* __restrict__ g, const int* __restrict__ tokens, const T* __restrict__ table, long long ldt,
+                                  int off, int dim, int ld, T* __restrict__ out, long long total) {
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long n = i / ld;
+    const int c = int(i - n * ld);
+    stf(out + i, c < dim ? gelu_tanh_f(ldf(g + i)) * ldf(table + tokens[n] * ldt + off + c) : 0.f);
+  }
+}
+
 __global__ void swiglu_bwd_kernel(const __nv_bfloat16* gu, const __nv_bfloat16* __restrict__ dh, __nv_bfloat16* dgu,
                                   long long M, int F) {
   const int vpr = F / 8;
@@ -269,6 +310,35 @@ int lt_clamped_glu(int fp32, const void* gu, void* h, long long M, int F, float 
   if (fp32) clamped_glu_kernel<float><<<grid_for(M * F, 256), 256, 0, st>>>(static_cast<const float*>(gu), static_cast<float*>(h), M, F, limit, slope);
   else if (F % 8 == 0) clamped_glu8_kernel<<<grid_for(M * (F / 8), 256), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(h), M, F, limit, slope);
   else clamped_glu_kernel<__nv_bfloat16><<<grid_for(M * F, 256), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(h), M, F, limit, slope);
+  LT_LAUNCH_CHECK();
+  return 0;
+}
+// act(gate) * up for rows [gate | up] of gu [M, 2 F]; act 1: GELU (tanh form), 2: SiLU; live nullptr, or the number of blocks of
+// block_rows rows to do (on the device).
+int lt_act_glu(int fp32, const void* gu, void* h, long long M, int F, int act, const int* live, int block_rows, void* stream) {
+  using namespace lt;
+  if (act < 1 || act > 2) return -int(kStatusBadArgument);
+  if (M == 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  using bf = __nv_bfloat16;
+  const bool v8 = !fp32 && F % 8 == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(h)) & 15) == 0;
+  if (fp32) act_glu_kernel<float, 1><<<grid_for(M * F, 256), 256, 0, st>>>(static_cast<const float*>(gu), static_cast<float*>(h), M, F, act, live, block_rows);
+  else if (v8) act_glu_kernel<bf, 8><<<grid_for(M * (F / 8), 256), 256, 0, st>>>(static_cast<const bf*>(gu), static_cast<bf*>(h), M, F, act, live, block_rows);
+  else act_glu_kernel<bf, 1><<<grid_for(M * F, 256), 256, 0, st>>>(static_cast<const bf*>(gu), static_cast<bf*>(h), M, F, act, live, block_rows);
+  LT_LAUNCH_CHECK();
+  return 0;
+}
+// g [n, ld] -> out [n, ld]; table [vocab, ldt].
+int lt_token_gate(int fp32, const void* g, const int* tokens, const void* table, long long ldt, int off, int dim, int ld, void* out,
+                  int n, void* stream) {
+  using namespace lt;
+  if (dim > ld) return -int(kStatusBadArgument);
+  const long long total = (long long)n * ld;
+  if (total == 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  using bf = __nv_bfloat16;
+  if (fp32) token_gate_kernel<float><<<grid_for(total, 256), 256, 0, st>>>(static_cast<const float*>(g), tokens, static_cast<const float*>(table), ldt, off, dim, ld, static_cast<float*>(out), total);
+  else token_gate_kernel<bf><<<grid_for(total, 256), 256, 0, st>>>(static_cast<const bf*>(g), tokens, static_cast<const bf*>(table), ldt, off, dim, ld, static_cast<bf*>(out), total);
   LT_LAUNCH_CHECK();
   return 0;
 }

@@ -267,7 +267,7 @@ int lt_window_attn(int fp32, const void* q, const void* k_cache, const void* v_c
                    int block_size, int window, float scale, void* stream) {
   using namespace lt;
   if (N == 0) return 0;
-  if (G < 1 || H % G != 0 || (DP & 3) || DP + EP > 2048) return -4;
+  if (G < 1 || H % G != 0 || (DP & 3) || DP + EP > 3072) return -4;
   const int smem = kWaWarps * (DP + EP) * 4;
   const long long items = (long long)N * H;
   const unsigned grid = unsigned((items + kWaWarps - 1) / kWaWarps);

@@ -63,8 +63,11 @@ def cuda_sources():
 
 # Sets of sources that a program which needs only a part of the library can build by themselves (`ensure_cuda`).
 COMPONENTS = {
-    "serving": ["common/host.cu", "gemm_sm100.cu", "gemm_skinny.cu", "gemv.cu", "flash_fwd.cu", "paged_decode.cu", "pointwise.cu"],
-    "hybrid": ["hyper_norm.cu", "gemm_simt.cu", "window_attn.cu", "rglru.cu", "mlstm.cu"],
+    "serving": ["common/host.cu", "gemm_sm100.cu", "gemm_skinny.cu", "gemv.cu", "flash_fwd.cu", "pointwise.cu"],
+    "paged": ["paged_decode.cu"],
+    "simt": ["gemm_simt.cu", "window_attn.cu"],
+    "hybrid": ["hyper_norm.cu", "rglru.cu", "mlstm.cu"],
+    "latent": ["residual_norm.cu", "latent_attn.cu", "moe_serve.cu"],
 }
 
 

@@ -194,6 +194,8 @@ class LatentAttentionWeights:
         big, small = (64 if latent_tc else 8), (64 if self.tensor_cores else 8)
         self.c, self.r = round_up(a.kv_rank, big), round_up(a.rot_dim, big)   # as in the cache: equal for all layers that share it
         self.d, self.v = round_up(a.dim, small), round_up(a.vdim, small)
+        if self.tensor_cores and self.d == 128:
+            self.v = 128                                                      # the kernel for the larger keys has one value size
         H = a.heads
         q = get(p + "q")
         W = q.shape[1]

@@ -119,7 +119,7 @@ def _serve_safuvik(engine, num_blocks, block_size, max_num_seqs, kv_dtype, graph
 
 
 register(ModelFamily("safuvik", lambda c: c.get("architecture") == "Safuvik", _load_safuvik, _is_safuvik_engine, _serve_safuvik,
-                     dtypes=(torch.bfloat16, torch.float32), components=("serving", "hybrid")))
+                     dtypes=(torch.bfloat16, torch.float32), components=("serving", "paged", "simt", "hybrid")))
 
 
 # ---------------------------------------------------------------------------------------------------- Ravenex
@@ -143,4 +143,4 @@ def _serve_ravenex(engine, num_blocks, block_size, max_num_seqs, kv_dtype, graph
 
 
 register(ModelFamily("ravenex", lambda c: c.get("architecture") == "Ravenex", _load_ravenex, _is_ravenex_engine, _serve_ravenex,
-                     dtypes=(torch.bfloat16, torch.float32), components=("serving", "hybrid", "latent")))
+                     dtypes=(torch.bfloat16, torch.float32), components=("serving", "simt", "latent")))

@@ -16,6 +16,18 @@ from .._native import cuda_lib
 _vp, _i, _ll, _f = c_void_p, c_int, c_longlong, c_float
 
 _SIGS = {
+    "lt_residual_norm": [_i, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _i, _vp, _f, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
+    "lt_latent_rope": [_i, _vp, _ll] + [_i] * 8 + [_vp, _f, _vp, _vp, _vp, _f, _vp, _i, _i, _vp, _vp, _vp],
+    "lt_latent_decode": [_vp] * 7 + [_i] * 8 + [_f, _vp],
+    "lt_flash_fwd_shared": [_vp] * 6 + [_i] * 5 + [_ll] * 4 + [_f, _i, _vp],
+    "lt_moe_plan": [_vp] * 12 + [_i] * 5 + [_vp],
+    "lt_moe_grouped_gemm": [_vp] * 5 + [_i] * 4 + [_vp],
+    "lt_gemm_skinny_glu": [_vp, _ll, _vp, _vp, _i, _i, _i, _i, _vp],
+    "lt_gemm_skinny_batch": [_vp, _ll, _ll, _vp, _vp, _ll, _ll, _i, _i, _i, _i, _vp],
+    "lt_gemm_skinny_grouped": [_vp, _ll] + [_vp] * 6 + [_i] * 5 + [_vp],
+    "lt_gemm_simt_grouped": [_i, _vp, _ll] + [_vp] * 6 + [_i] * 3 + [_vp],
+    "lt_act_glu": [_i, _vp, _vp, _ll, _i, _i, _vp, _i, _vp],
+    "lt_token_gate": [_i, _vp, _vp, _vp, _ll, _i, _i, _i, _vp, _i, _vp],
     "lt_flash_fwd_window": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _ll, _ll, _ll, _ll, _ll, _ll, _ll, _ll, _f, _i, _vp],
     "lt_paged_decode_window": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _f, _i, _vp, _ll, _i, _vp],
     "lt_clamped_glu": [_i, _vp, _vp, _ll, _i, _f, _f, _vp],
@@ -109,7 +121,7 @@ _SIGS = {
 _bound = {}
 
 # Kernels launched per native call; `launch_count()` is what bench.py reports as "gpu_launches".
-_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_paged_decode_window": 2, "lt_mlstm_prefill": 4, "lt_rglru_scan": 3, "lt_rglru_step": 2, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
+_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_paged_decode_window": 2, "lt_latent_decode": 2, "lt_mlstm_prefill": 4, "lt_rglru_scan": 3, "lt_rglru_step": 2, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
                       "lt_adam_chunk_elems": 0}
 _launches = [0]
 
@@ -879,10 +891,11 @@ def qkv_rope(proj, q_off: int, k_off: int, v_off: int, H: int, G: int, D: int, E
 
 
 def kv_gather(k_cache, v_cache, table, pos0: int, n: int, k_lin, v_lin):
-    """Keys and values of positions pos0 .. pos0 + n - 1 of the sequence with block table `table` into k_lin / v_lin [n, G, .]."""
-    rc = _fn("lt_kv_gather")(k_cache.data_ptr(), v_cache.data_ptr(), k_lin.data_ptr(), v_lin.data_ptr(), table.data_ptr(), pos0, n,
-                             k_cache.shape[1], k_cache.shape[3] * k_cache.element_size(), v_cache.shape[3] * v_cache.element_size(),
-                             k_cache.shape[2], _stream())
+    """Keys and values of positions pos0 .. pos0 + n - 1 of the sequence with block table `table` into k_lin / v_lin [n, G, .]
+    (v_cache and v_lin None: a cache without values)."""
+    rc = _fn("lt_kv_gather")(k_cache.data_ptr(), _p(v_cache), k_lin.data_ptr(), _p(v_lin), table.data_ptr(), pos0, n,
+                             k_cache.shape[1], k_cache.shape[3] * k_cache.element_size(),
+                             0 if v_cache is None else v_cache.shape[3] * v_cache.element_size(), k_cache.shape[2], _stream())
     _check(rc, "lt_kv_gather")
 
 
@@ -995,6 +1008,220 @@ def head_norm_gate(o, w, gate, H: int, eps: float):
     rc = _fn("lt_head_norm_gate")(_f32(out), o.data_ptr(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), R, H, HE // H,
                                   float(eps), _stream())
     _check(rc, "lt_head_norm_gate")
+    return out
+
+
+# ------------------------------------------------------------------------------------------------ latent attention, experts
+# As above: bf16 or fp32 activations.
+_ACT = {"gelu": 1, "silu": 2}
+
+
+def _aligned(*ts) -> bool:
+    return all(t.data_ptr() % 16 == 0 for t in ts)
+
+
+def residual_norm(x, eps: float, *, dtype, norm=None, mult: float = 1.0, y=None, y_norm=None, experts=None, tokens=None, embed=None,
+                  rows=None, write=True):
+    """One step along a single residual x [T, W] (fp32, updated in place): x += mult * (RMS norm of the finished sublayer's output,
+    weighted with y_norm; None: the output itself), then returns the RMS norm of x weighted with `norm` (None: x itself) as
+    [rows, W] of `dtype`.  The output is y [T, W], or the weighted sum of a token's expert rows - experts = (z [., W],
+    slots [T, k], weights [T, k]) - or their sum.  With `embed` the residual starts as embed[tokens]; `rows` picks tokens;
+    write=False leaves x alone."""
+    T, W = x.shape
+    n = T if rows is None else rows.shape[0]
+    h = torch.empty((n, W), dtype=dtype, device=x.device)
+    z, slots, weight = experts if experts is not None else (None, None, None)
+    assert x.is_contiguous() and x.dtype == torch.float32 and all(t is None or t.dtype == dtype for t in (y, z, embed))
+    assert y is None or y.stride(1) == 1
+    assert z is None or (z.is_contiguous() and slots.is_contiguous() and weight.is_contiguous())
+    rc = _fn("lt_residual_norm")(_f32(h), x.data_ptr(), _p(tokens), _p(embed), _p(y), y.stride(0) if y is not None else 0, _p(z), _p(slots),
+                                 _p(weight), slots.shape[1] if slots is not None else 0, _p(y_norm), float(mult), _p(norm), float(eps),
+                                 h.data_ptr(), _p(rows), n, W, 1 if write else 0, _stream())
+    _check(rc, "lt_residual_norm")
+    return h
+
+
+def latent_rope(proj, H: int, d: int, r: int, rot: int, positions, slots, *, freq, gain: float = 1.0, c_off: int = -1, rank: int = 0,
+                c_norm=None, eps: float = 1e-6, cache=None, q_out=None, lin=None):
+    """Takes a latent-attention layer's fused projection [N, H (d + r) | latent (rank), key part (rot)]: rotates the last part of every
+    head's query (interleaved pairs, angle position * freq[i]) in place, or into the last r columns of q_out [N, H, .], with
+    c_off >= 0 also norms the latent, rotates the key part and writes both, each padded with zeros, to the rows `slots` of the
+    paged cache [blocks, 1, block size, c + r] (and, one after another, to lin [N, c + r])."""
+    N = proj.shape[0]
+    assert proj.stride(1) == 1 and (q_out is None or q_out.is_contiguous()) and (lin is None or lin.is_contiguous())
+    width = cache.shape[3] if c_off >= 0 else 0
+    rc = _fn("lt_latent_rope")(_f32(proj), proj.data_ptr(), proj.stride(0), N, H, d, r, rot, c_off, rank, width - r if c_off >= 0 else 0, _p(c_norm),
+                               float(eps), positions.data_ptr(), slots.data_ptr(), freq.data_ptr(), float(gain), _p(q_out),
+                               q_out.shape[2] if q_out is not None else 0, q_out.shape[2] - r if q_out is not None else 0,
+                               _p(cache) if c_off >= 0 else None, _p(lin), _stream())
+    _check(rc, "lt_latent_rope")
+
+
+def head_linear(x, w, out=None):
+    """y[n, h] = w[h] @ x[n, h] for x [N, H, K] and w [H, M, K]: a product per head.  x and out may be strided views."""
+    (N, H, Kd), M = x.shape, w.shape[1]
+    y = torch.empty((N, H, M), dtype=x.dtype, device=x.device) if out is None else out
+    assert x.stride(2) == 1 and y.stride(2) == 1 and w.is_contiguous() and w.shape == (H, M, Kd) and x.dtype == w.dtype == y.dtype
+    if (x.dtype == torch.bfloat16 and Kd % 32 == 0 and M % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0 and y.stride(0) % 2 == 0
+            and y.stride(1) % 2 == 0 and _aligned(x, w) and y.data_ptr() % 4 == 0):
+        for n in range(0, N, 128):
+            rc = _fn("lt_gemm_skinny_batch")(x[n:].data_ptr(), x.stride(0), x.stride(1), w.data_ptr(), y[n:].data_ptr(), y.stride(0), y.stride(1), H,
+                                             min(128, N - n), M, Kd, _stream())
+            _check(rc, "lt_gemm_skinny_batch")
+        return y
+    rc = _fn("lt_gemm_simt")(_f32(x), _f32(y), x.data_ptr(), w.data_ptr(), y.data_ptr(), N, M, Kd, x.stride(0), Kd, y.stride(0), H, x.stride(1),
+                             M * Kd, y.stride(1), 1.0, _stream())
+    _check(rc, "lt_gemm_simt")
+    return y
+
+
+def shared_rope_fwd(q, k, k_rot, v, *, scale: float, window: int = 0):
+    """Causal attention of one sequence, the last query on the last key, with keys in two parts: q [n, H, D], k [T, H, D - 64], k_rot
+    [T, 64] (the last 64 columns of every head's keys), v [T, H, DV] -> [n, H, DV].  Rows may be strided, heads are packed.
+    window > 0: a query sees its own position and the window - 1 before it."""
+    (n, H, D), (T, _, DV) = q.shape, v.shape
+    for t in (q, k, v):
+        assert t.stride(2) == 1 and t.stride(1) == t.shape[2] and t.dtype == torch.bfloat16
+    assert k.shape == (T, H, D - 64) and k_rot.shape == (T, 64) and k_rot.stride(1) == 1
+    o = torch.empty((n, H, DV), dtype=q.dtype, device=q.device)
+    lse = torch.empty((H, n), dtype=torch.float32, device=q.device)
+    rc = _fn("lt_flash_fwd_shared")(q.data_ptr(), k.data_ptr(), k_rot.data_ptr(), v.data_ptr(), o.data_ptr(), lse.data_ptr(), n, T, H, D, DV,
+                                    q.stride(0), k.stride(0), k_rot.stride(0), v.stride(0), float(scale), int(window), _stream())
+    _check(rc, "lt_flash_fwd_shared")
+    return o
+
+
+def latent_splits(S: int, H: int, keys: int, sms: int = 148) -> int:
+    """Splits of the key range per sequence: as few rounds of tiles over the SMs (one CTA each) as possible; a split costs about
+    two tiles on top of its own."""
+    ctas = S * ((H + 31) // 32)
+    best, cost = 1, None
+    for n in range(1, max(1, min(64, (keys + 63) // 64)) + 1):
+        waves = (ctas * n + sms - 1) // sms
+        c = waves * ((keys + 64 * n - 1) // (64 * n) + 2) + (2 if n > 1 else 0)
+        if cost is None or c < cost:
+            best, cost = n, c
+    return best
+
+
+def latent_decode(q, cache, tables, ctx, *, rank: int, window: int, scale: float, max_keys: int, splits: int = 0):
+    """Attention of q [S, H, w] over the rows of each sequence's pages (cache [blocks, 1, block size, w]): keys are the whole rows,
+    values their first `rank` columns; window > 0: the newest `window` of the ctx[s] rows.  Returns [S, H, rank]."""
+    S, H, w = q.shape
+    assert q.is_contiguous() and cache.is_contiguous() and cache.shape[1] == 1 and cache.shape[3] == w and q.dtype == cache.dtype == torch.bfloat16
+    splits = splits or latent_splits(S, H, max_keys)
+    o = torch.empty((S, H, rank), dtype=q.dtype, device=q.device)
+    part = torch.empty(S * H * splits * (rank + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
+    rc = _fn("lt_latent_decode")(q.data_ptr(), cache.data_ptr(), tables.data_ptr(), ctx.data_ptr(), _p(part),
+                                 part[S * H * splits * rank:].data_ptr() if splits > 1 else None, o.data_ptr(), S, H, rank, w, cache.shape[2],
+                                 tables.shape[1], splits, int(window), float(scale), _stream())
+    _check(rc, "lt_latent_decode")
+    return o
+
+
+def act_glu(gu, act: str, live=None, block_rows: int = 0):
+    """act(gate) * up for rows [gate | up]; live: a device count of blocks of block_rows rows that matter."""
+    M, F = gu.shape[0], gu.shape[1] // 2
+    h = torch.empty((M, F), dtype=gu.dtype, device=gu.device)
+    rc = _fn("lt_act_glu")(_f32(gu), gu.data_ptr(), h.data_ptr(), M, F, _ACT[act], _p(live), block_rows, _stream())
+    _check(rc, "lt_act_glu")
+    return h
+
+
+def glu_mlp(x, gu, down, act: str):
+    """down @ (act(gate @ x) * (up @ x)) with gu = [gate; up]; up to 128 rows of bf16 gate in the product's epilogue."""
+    M, Kd = x.shape
+    F = gu.shape[0] // 2
+    if x.dtype == torch.bfloat16 and 0 < M <= 128 and Kd % 32 == 0 and F % 8 == 0 and x.stride(0) % 8 == 0 and _aligned(x, gu):
+        h = torch.empty((M, F), dtype=x.dtype, device=x.device)
+        rc = _fn("lt_gemm_skinny_glu")(x.data_ptr(), x.stride(0), gu.data_ptr(), h.data_ptr(), M, F, Kd, _ACT[act], _stream())
+        _check(rc, "lt_gemm_skinny_glu")
+        return linear(h, down)
+    return linear(act_glu(linear(x, gu), act), down)
+
+
+def moe_plan(logits, correction, top: int, block_rows: int, x=None):
+    """The router's choice and the experts' slots for logits [N, E] (fp32): scores are sigmoids, the `top` with the largest score +
+    correction are chosen, a chosen expert's weight is its score.  Every expert owns whole blocks of block_rows slots.
+    Returns a dict: weight, slot [N, top]; src (token of a slot), group (expert of a block), rows (of the block in use), live
+    (blocks in use), blocks (bound of live), and - with x [N, W], more than 64 tokens - xs [slots, W], the tokens' rows in slots."""
+    N, E = logits.shape
+    dev = logits.device
+    assert logits.dtype == torch.float32 and logits.is_contiguous() and (x is None or (N > 64 and x.is_contiguous()))
+    blocks = min(N * top, E) + N * top // block_rows
+    i32 = lambda *s: torch.empty(s, dtype=torch.int32, device=dev)
+    p = dict(weight=torch.empty((N, top), dtype=torch.float32, device=dev), slot=i32(N, top), group=i32(blocks), rows=i32(blocks), live=i32(1),
+             src=i32(blocks * block_rows), blocks=blocks, block_rows=block_rows)
+    pairs = counts = None
+    if N > 64:
+        pairs, counts = i32(2 * N * top), torch.zeros(E, dtype=torch.int32, device=dev)
+    if x is not None:
+        p["xs"] = torch.empty((blocks * block_rows, x.shape[1]), dtype=x.dtype, device=dev)
+    rc = _fn("lt_moe_plan")(logits.data_ptr(), correction.data_ptr(), p["weight"].data_ptr(), p["slot"].data_ptr(), p["src"].data_ptr(),
+                            p["group"].data_ptr(), p["rows"].data_ptr(), p["live"].data_ptr(), _p(pairs), _p(counts), _p(x), _p(p.get("xs")),
+                            x.shape[1] * x.element_size() if x is not None else 0, N, E, top, block_rows, _stream())
+    _check(rc, "lt_moe_plan")
+    return p
+
+
+def moe_grouped(x, w, plan, act: str = "", picked: bool = False):
+    """Slots times their expert's matrix: x [slots, K] (or tokens, with picked=True: the plan's src picks the rows), w [experts, N, K];
+    with act, w holds gate and up rows and the result is gated.  The kernel follows from the plan's block size."""
+    E, N, Kd = w.shape
+    M = plan["blocks"] * plan["block_rows"]
+    dev, br = x.device, plan["block_rows"]
+    assert x.stride(1) == 1 and w.is_contiguous() and x.dtype == w.dtype and x.shape[1] == Kd
+    src = plan["src"] if picked else None
+    if br == 128:
+        assert x.is_contiguous() and not picked
+        y = torch.empty((M, N), dtype=x.dtype, device=dev)
+        rc = _fn("lt_moe_grouped_gemm")(x.data_ptr(), w.data_ptr(), y.data_ptr(), plan["group"].data_ptr(), plan["live"].data_ptr(), plan["blocks"], E, N,
+                                        Kd, _stream())
+        _check(rc, "lt_moe_grouped_gemm")
+        return act_glu(y, act, plan["live"], br) if act else y
+    if x.dtype == torch.bfloat16 and plan["mma"]:
+        n = N // 2 if act else N
+        y = torch.empty((M, n), dtype=x.dtype, device=dev)
+        rc = _fn("lt_gemm_skinny_grouped")(x.data_ptr(), x.stride(0), w.data_ptr(), y.data_ptr(), plan["group"].data_ptr(), plan["rows"].data_ptr(),
+                                           plan["live"].data_ptr(), _p(src), plan["blocks"], br, n, Kd, _ACT[act] if act else 0, _stream())
+        _check(rc, "lt_gemm_skinny_grouped")
+        return y
+    assert br == 64
+    y = torch.empty((M, N), dtype=x.dtype, device=dev)
+    rc = _fn("lt_gemm_simt_grouped")(_f32(x), x.data_ptr(), x.stride(0), w.data_ptr(), y.data_ptr(), plan["group"].data_ptr(), plan["rows"].data_ptr(),
+                                     plan["live"].data_ptr(), _p(src), plan["blocks"], N, Kd, _stream())
+    _check(rc, "lt_gemm_simt_grouped")
+    return act_glu(y, act, plan["live"], br) if act else y
+
+
+def moe_logits(x, router):
+    """The router's logits as fp32."""
+    return rows_dot(x, router) if x.shape[0] <= 64 else linear(x, router, out_dtype=torch.float32)
+
+
+def moe_experts(x, router, correction, top: int, gu, down, act: str):
+    """x [N, W] through the `top` experts of every token (gu [experts, 2 F, W], down [experts, W, F]): the expert rows in slots, and
+    every token's slots and weights, as `residual_norm` takes them."""
+    N, W = x.shape
+    E, F = gu.shape[0], gu.shape[1] // 2
+    logits = moe_logits(x, router)
+    mean = N * top / E                                    # rows an expert gets
+    mma = x.dtype == torch.bfloat16 and W % 32 == 0 and F % 32 == 0 and _aligned(x, gu, down)
+    if mma and mean > 48 and N > 64:
+        plan = moe_plan(logits, correction, top, 128, x)
+        return moe_grouped(moe_grouped(plan["xs"], gu, plan, act), down, plan), plan["slot"], plan["weight"]
+    plan = moe_plan(logits, correction, top, 64 if not mma or mean > 24 else 32 if mean > 12 else 16)
+    plan["mma"] = mma
+    return moe_grouped(moe_grouped(x, gu, plan, act, picked=True), down, plan), plan["slot"], plan["weight"]
+
+
+def token_gate(g, tokens, table, off: int, dim: int):
+    """gelu(g [N, F]) * table[tokens, off : off + dim], zeros from column dim on."""
+    assert g.is_contiguous() and table.is_contiguous() and table.dtype == g.dtype
+    out = torch.empty_like(g)
+    rc = _fn("lt_token_gate")(_f32(g), g.data_ptr(), tokens.data_ptr(), table.data_ptr(), table.shape[1], off, dim, g.shape[1], out.data_ptr(),
+                              g.shape[0], _stream())
+    _check(rc, "lt_token_gate")
     return out
 
 
