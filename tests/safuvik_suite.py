@@ -1,14 +1,9 @@
-"""Small Safuvik models and comparisons shared by the CPU and the GPU tests: the framework's sessions, scheduler and
-generation against the plain statement in `safuvik_ref`."""
-import json
-import os
-
+"""Small Safuvik models for the CPU and the GPU tests, compared with the plain statement in `safuvik_ref`."""
 import torch
 
 import safuvik_ref as R
-from litetorch_b200.models import registry
+from decoder_suite import ServingScheduler, Suite, error, run_portions, server, tokens, write_model          # noqa: F401  (used through this module)
 from litetorch_b200.models.safuvik import SafuvikConfig, SafuvikEngine, random_tensor, tensor_shapes
-from litetorch_b200.serving import Request, ServingScheduler
 
 
 def attention(heads, kv, dim, vdim, window, dims, scale=None, base=700.0, yarn=None):
@@ -71,124 +66,9 @@ def engine(cfg, w, device, dtype):
     return SafuvikEngine(SafuvikConfig.parse(cfg), w, device, dtype)
 
 
-def tokens(cfg, n, seed):
-    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def server(eng, blocks=64, slots=4, block_size=16):
-    return registry.new_serving(eng, num_blocks=blocks, block_size=block_size, max_num_seqs=slots), ServingScheduler(blocks, block_size, slots, 4096, -1)
-
-
-def reference(cfg, w, toks):
-    with torch.no_grad():
-        return R.forward(cfg, w, toks)
-
-
-def error(got, want):
-    """How far rows of logits are from what they should be (means taken off), relative to the size of all of them: the larger
-    of the root mean square over the rows and a third of the worst row."""
-    dlt = got.double().cpu() - want
-    dlt = dlt - dlt.mean(-1, keepdim=True)
-    row = dlt.pow(2).mean(-1) / want.var()
-    return max(float(row.mean().sqrt()), float(row.max().sqrt()) / 3.0)
-
-
-def run_portions(model, sched, sid, toks, cuts):
-    """Feed a sequence in portions of the given sizes (the last one repeats); logits at every position."""
-    out, at, k = [], 0, 0
-    while at < len(toks):
-        n = min(cuts[min(k, len(cuts) - 1)], len(toks) - at)
-        out.append(sched.feed(model, [(sid, toks[at:at + n], list(range(n)))])[0])
-        at += n
-        k += 1
-    return torch.cat(out)
-
-
-TOL = {torch.float32: 1e-5, torch.bfloat16: 0.03}
-
-
-def check_portions(name, device, dtype, length, schedules):
-    """Whole prompts, portions and single tokens all give the logits of the plain statement."""
-    cfg = CONFIGS[name]
-    w = weights(cfg)
-    toks = tokens(cfg, length, 1)
-    want = reference(cfg, w, toks)
-    model, sched = server(engine(cfg, w, device, dtype), blocks=2 * (length // 16 + 2))
-    for n, cuts in enumerate(schedules):
-        e = error(run_portions(model, sched, n, toks, cuts), want)
-        assert e < TOL[dtype], (name, cuts, e)
-        sched.end_session(n)
-
-
-def check_interleaved(name, device, dtype):
-    """Requests of unequal lengths in one step, prompts beside decoding, each against itself alone; then the pages and
-    slots they leave are used by others."""
-    cfg = CONFIGS[name]
-    w = weights(cfg, 3)
-    model, sched = server(engine(cfg, w, device, dtype), blocks=40, slots=4)
-    free = sched.free_blocks
-    for rnd in range(2):                                     # the second round meets the first one's cache and state
-        lens = [70, 9, 41, 100] if rnd == 0 else [12, 97, 60, 33]
-        seqs = [tokens(cfg, n, 10 * rnd + i) for i, n in enumerate(lens)]
-        want = [reference(cfg, w, s) for s in seqs]
-        at, got = [0] * 4, [[] for _ in range(4)]
-        step = 0
-        while any(at[i] < lens[i] for i in range(4)):
-            entries = []
-            for i in range(4):
-                n = min([1, 1, 5, 1, 2, 1, 17][(step + 2 * i) % 7] if step else lens[i] // 3, lens[i] - at[i])
-                if n:
-                    entries.append((100 + i, seqs[i][at[i]:at[i] + n], list(range(n))))
-                    at[i] += n
-            for (sid, _, _), y in zip(entries, sched.feed(model, entries)):
-                got[sid - 100].append(y.cpu())
-            step += 1
-        for i in range(4):
-            e = error(torch.cat(got[i]), want[i])
-            assert e < TOL[dtype], (name, rnd, i, e)
-            sched.end_session(100 + i)
-        assert sched.free_blocks == free
-
-
-def check_generate(name, device, dtype, max_new, budget):
-    """Greedy generation through the scheduler: every token is the argmax of the plain statement's logits, up to rounding."""
-    from litetorch_b200.models.serving_base import generate
-    cfg = CONFIGS[name]
-    w = weights(cfg, 5)
-    prompts = [tokens(cfg, n, 40 + n) for n in (1, 2, 30, 75)]
-    outs = generate(engine(cfg, w, device, dtype), prompts, max_new, max_num_seqs=3, max_num_batched_tokens=budget)
-    for p, o in zip(prompts, outs):
-        assert len(o) == max_new
-        y = reference(cfg, w, p + o[:-1])[len(p) - 1:]
-        gap = y.max(-1).values - y[torch.arange(max_new), torch.tensor(o)]
-        assert float(gap.max() / y.std()) < 5 * TOL[dtype], (name, len(p), float(gap.max()))
+SUITE = Suite(CONFIGS, weights, engine, R.forward)
+reference, check_portions, check_interleaved, check_generate = SUITE.reference, SUITE.check_portions, SUITE.check_interleaved, SUITE.check_generate
 
 
 def check_generate_matches_decode_of_requests(device, dtype):
-    """Requests that join and leave a running batch of the scheduler see each other in nothing."""
-    cfg = CONFIGS["mixed"]
-    w = weights(cfg, 6)
-    eng = engine(cfg, w, device, dtype)
-
-    def run(prompts, slots):
-        model = registry.new_serving(eng, num_blocks=64, max_num_seqs=slots)
-        sched = ServingScheduler(64, 16, slots, 24, -1)
-        reqs = [Request(i, p, max_new_tokens=4 + 3 * i) for i, p in enumerate(prompts)]
-        for r in reqs:
-            sched.add_request(r)
-        done = []
-        while len(done) < len(reqs):
-            done += sched.step(model)
-        assert sched.free_blocks == 64
-        return [r.generated_tokens for r in reqs]
-
-    prompts = [tokens(cfg, n, n) for n in (50, 3, 21, 34, 8)]
-    assert run(prompts, 2) == run(prompts, 5)
-
-
-def write_model(directory, cfg, w):
-    from safetensors.torch import save_file
-    os.makedirs(directory, exist_ok=True)
-    save_file({k: v.contiguous() for k, v in w.items()}, os.path.join(directory, "model.safetensors"))
-    with open(os.path.join(directory, "config.json"), "w") as f:
-        json.dump(cfg, f)
+    SUITE.check_generate_matches_decode_of_requests("mixed", device, dtype)
