@@ -57,9 +57,9 @@ def _parse():
     ap.add_argument("--hybrid", action="store_true",
                     help="with --tp 1: shard over dp with the FSDP x TP provider (weights prefetched by peer-pull kernels) "
                          "instead of the ZeRO-3 provider whose all-gather runs inside the GEMMs")
-    ap.add_argument("--serving-compare", action="store_true",
-                    help="instead of the training workload: prompt and decode throughput of Safuvik models beside Llama models of equal "
-                         "size, and their kernels (litetorch_b200.utils.hybrid_bench; prints JSON lines and tables)")
+    ap.add_argument("--serving-compare", nargs="?", const="safuvik", choices=["safuvik", "ravenex"],
+                    help="instead of the training workload: prompt and decode throughput of the named design beside Llama models of equal "
+                         "size, and their kernels (litetorch_b200.utils.hybrid_bench / latent_bench; prints JSON lines and tables)")
     return ap.parse_args()
 
 
@@ -424,8 +424,8 @@ def run_reference(args):
 if __name__ == "__main__":
     a = _parse()
     if a.serving_compare:
-        from litetorch_b200.utils import hybrid_bench
-        hybrid_bench.main([])
+        from litetorch_b200.utils import hybrid_bench, latent_bench
+        (latent_bench if a.serving_compare == "ravenex" else hybrid_bench).main([])
     elif a.impl == "reference":
         run_reference(a)
     else:
