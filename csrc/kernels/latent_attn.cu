@@ -8,6 +8,7 @@
 //   latent_decode_kernel   split-K decode attention of up to 32 heads per CTA on the rows of a sequence's pages
 //   latent_merge_kernel    combines the splits
 #include "lt_cuda.h"
+#include <cuda.h>
 #include "common/host.h"
 #include "common/ptx.cuh"
 #include "common/scalar.cuh"
@@ -94,24 +95,30 @@ __global__ void __launch_bounds__(kRopeThreads) latent_rope_kernel(const RopePar
 }
 
 // ------------------------------------------------------------------------------------------------------------ decode
-// One CTA of eight warps per (sequence, group of up to 16 MT heads, split of the visible keys).  Tiles of 64 rows arrive by
-// plain bulk copies, one per row (rows of a sequence lie in pages), at a pitch of 16 bytes more than a row, so that
-// ldmatrix meets no bank conflicts; a ring of `stages` tiles is filled ahead.  Per tile:
-//   scores   warp = 16 keys x one half of the c + r columns (mma.sync m16n8k16: heads x keys), halves added through shared
-//            memory; the query block stays in shared memory
+// One CTA per (sequence, group of up to 16 MT heads, split of the visible keys): eight warps make scores and weights, eight
+// more the values, one tile of 32 rows behind.  Tiles arrive by TMA tensor copies, one per page (issuing a copy costs its warp
+// on the order of a hundred cycles, so rows or 64-column panels one by one would bound the kernel): the map sees a row as panels
+// of 64 columns, and a copy lands as [panel][row][64 columns] in the 128-byte-swizzled layout, so that ldmatrix meets no bank
+// conflicts.  Per tile:
+//   scores   warp = 16 keys x a quarter of the c + r columns (mma.sync m16n8k16: heads x keys), the quarters added through
+//            shared memory; a warp's part of the query block stays in its registers
 //   softmax  256 / (16 MT) threads per head: running maximum and sum in registers, weights as bf16 operands to shared
 //   values   warp = an eighth of the c columns: accumulators in registers, rows read transposed from the same tile
-// tcgen05 is not the tool here: its 64- or 128-row tiles would be mostly empty at 16 or 32 heads, 512 value columns of them
-// would fill the tensor memory, and the kernel is bound by streaming the rows.
-constexpr int kLdThreads = 256;
-constexpr int kLdKeys = 64;
-constexpr int kLdMaxStages = 4;
-constexpr int kLdSPitch = kLdKeys + 4;      // floats
+// mbarriers hand over tiles (ring of `stages`), weights (two buffers) and both back.  A second kernel merges the splits (measured:
+// quicker than merging them as a thread-block cluster through distributed shared memory).
+// tcgen05 is not used: with 16 or 32 heads its 128-row tiles would be mostly empty, and 512 value columns of them would fill
+// the tensor memory.
+constexpr int kLdThreads = 512;
+constexpr int kLdRole = 256;                // threads of each half
+constexpr int kLdKeys = 32;
+constexpr int kLdMaxStages = 6;
+constexpr int kLdMaxSplits = 64;
+constexpr int kLdMaxKs = 9;                 // 16-column steps of a quarter: w up to 576
+constexpr int kLdSPitch = kLdKeys + 8;      // floats
 constexpr int kLdPPitch = kLdKeys + 8;      // bf16
 
 struct LatentDecodeParams {
-  const __nv_bfloat16* q;        // [S, H, w]
-  const __nv_bfloat16* cache;    // [rows, w], w = c + r, a multiple of 64
+  const __nv_bfloat16* q;        // [S, H, w], w = c + r, a multiple of 64
   const int* tables;             // [S, max_blocks]
   const int* ctx;                // [S] keys of the sequence, the query's own included
   float* part;                   // [S * H, splits, c] unnormalised outputs
@@ -136,32 +143,41 @@ __device__ __forceinline__ void ld_mma(float (&d)[4], const uint32_t (&a)[4], ui
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void ld_bulk(uint32_t smem_dst, const void* gsrc, uint32_t bytes, uint32_t bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-               ::"r"(smem_dst), "l"(gsrc), "r"(bytes), "r"(bar) : "memory");
+// Barriers of the eight warps that make the scores.
+__device__ __forceinline__ bool ld_bar_and(bool v) {
+  int r;
+  asm volatile("{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbar.red.and.pred q, 1, 256, p;\nselp.s32 %0, 1, 0, q;\n}" : "=r"(r) : "r"(int(v)) : "memory");
+  return r != 0;
 }
 
-// Shared memory of a CTA: tiles, query block, score halves, weights, per-head factors, barriers.
+// Shared memory of a CTA: slack for alignment, tiles (later the outputs of the split), score quarters, weights, per-head numbers,
+// barriers.
 __host__ __device__ inline int ld_smem_bytes(int w, int heads, int stages) {
-  const int pitch = w * 2 + 16;
-  return stages * kLdKeys * pitch + heads * pitch + 2 * heads * kLdSPitch * 4 + heads * kLdPPitch * 2 + 3 * heads * 4 + kLdMaxStages * 8 + 16;
+  return 1024 + stages * kLdKeys * w * 2 + 2 * (4 * heads * kLdSPitch * 4 + heads * kLdPPitch * 2 + heads * 4) + 2 * heads * 4 +
+         (2 * kLdMaxStages + 4) * 8;
 }
 
-// MT: 16-head blocks of a CTA (1 or 2).
-template <int MT>
-__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LatentDecodeParams p) {
+// MT: 16-head blocks of a CTA (1 or 2).  FULL: the largest row (w 576, c 512),
+// whose loops have no conditions, so that loads run ahead of the products.
+template <int MT, bool FULL>
+__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap tmap,
+                                                                               const LatentDecodeParams p) {
   constexpr int MH = MT * 16;
-  constexpr int TPH = kLdThreads / MH;           // threads per head in the softmax
+  constexpr int TPH = kLdRole / MH;              // threads per head in the softmax
   constexpr int KPT = kLdKeys / TPH;             // keys of each
-  extern __shared__ __align__(128) uint8_t ld_smem[];
-  const int pitch = p.w * 2 + 16, tile_bytes = kLdKeys * pitch;
-  uint8_t* q_s = ld_smem + p.stages * tile_bytes;
-  float* s_s = reinterpret_cast<float*>(q_s + MH * pitch);                             // [2][MH][kLdSPitch]
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_s + 2 * MH * kLdSPitch);     // [MH][kLdPPitch]
-  float* f_s = reinterpret_cast<float*>(p_s + MH * kLdPPitch);                         // [MH] rescale of the tile
-  float* m_s = f_s + MH;                                                               // [MH] final maximum, then sum
+  extern __shared__ uint8_t ld_raw[];
+  uint8_t* ld_smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ld_raw) + 1023) & ~uintptr_t(1023));
+  const int tile_bytes = kLdKeys * p.w * 2;
+  float* s_s = reinterpret_cast<float*>(ld_smem + p.stages * tile_bytes);              // [2][4][MH][kLdSPitch]
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_s + 2 * 4 * MH * kLdSPitch); // [2][MH][kLdPPitch]
+  float* f_s = reinterpret_cast<float*>(p_s + 2 * MH * kLdPPitch);                     // [2][MH] rescale of the tile
+  float* m_s = f_s + 2 * MH;                                                           // [MH] final maximum, then sum
   float* l_s = m_s + MH;
   const uint32_t bars = smem_u32(l_s + MH);
+  auto full = [&](int st) { return bars + 8u * st; };                                  // the tile has arrived
+  auto empty = [&](int st) { return bars + 8u * (kLdMaxStages + st); };                // nobody needs the tile any more
+  auto p_full = [&](int b) { return bars + 8u * (2 * kLdMaxStages + b); };             // weights and rescale factors are there
+  auto p_free = [&](int b) { return bars + 8u * (2 * kLdMaxStages + 2 + b); };
   __shared__ int abort_s, drain_s;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -169,190 +185,260 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
   const int heads = min(MH, p.H - h0);
   const int ctx = p.ctx[s];
   const int lo = p.window > 0 ? max(0, ctx - p.window) : 0;
-  const int per = ((ctx - lo + p.splits - 1) / p.splits + kLdKeys - 1) / kLdKeys * kLdKeys;
-  const int t0 = lo + sp * per, t1 = min(ctx, t0 + per);
-  if (t0 >= t1) {                                // nothing left for this split
-    if (threadIdx.x < heads) {
-      float* st = p.stat + (((long long)s * p.H + h0 + threadIdx.x) * p.splits + sp) * 2;
-      st[0] = -INFINITY;
-      st[1] = 0.f;
-    }
-    return;
-  }
-  const int tiles = (t1 - t0 + kLdKeys - 1) / kLdKeys;
-  const int* bt = p.tables + (long long)s * p.max_blocks;
+  const int base = lo & ~(kLdKeys - 1);          // tiles start on multiples of 32 keys, and so on a page or its half, quarter, ..
+  const int per = ((ctx - base + p.splits - 1) / p.splits + kLdKeys - 1) / kLdKeys * kLdKeys;
+  const int t0 = base + sp * per, t1 = min(ctx, t0 + per);
+  const int tiles = t1 > t0 ? (t1 - t0 + kLdKeys - 1) / kLdKeys : 0;      // 0: nothing left for this split
+  const int run = min(p.block_size, kLdKeys), run_log = 31 - __clz(run), panels = p.w / 64, run_bytes = run * panels * 128;
+  // where 16-byte unit u of row r of a tile lies
+  auto unit_at = [&](int r, int u) {
+    return (r >> run_log) * run_bytes + ((((u >> 3) << run_log) + (r & (run - 1))) << 7) + (((u & 7) ^ (r & 7)) << 4);
+  };
   if (threadIdx.x == 0) {
     abort_s = 0; drain_s = 0;
-    for (int i = 0; i < p.stages; ++i) mbar_init(bars + 8u * i, 1);
+    for (int i = 0; i < p.stages; ++i) { mbar_init(full(i), 1); mbar_init(empty(i), kLdRole / 32); }
+    for (int b = 0; b < 2; ++b) { mbar_init(p_full(b), kLdRole / 32); mbar_init(p_free(b), kLdRole / 32); }
     fence_barrier_init();
     fence_proxy_async();
   }
-  {
-    const int units = p.w / 8;
-    const __nv_bfloat16* q = p.q + ((long long)s * p.H + h0) * p.w;
-    for (int i = threadIdx.x; i < MH * units; i += kLdThreads) {
-      const int h = i / units, u = i - h * units;
-      *reinterpret_cast<uint4*>(q_s + h * pitch + u * 16) =
-          h < heads ? *reinterpret_cast<const uint4*>(q + (long long)h * p.w + u * 8) : make_uint4(0u, 0u, 0u, 0u);
-    }
-  }
   __syncthreads();
   volatile int* abort_flag = &abort_s;
-  // the rows of tile i into its stage, two per lane of warp 0; past the last key that key's row again (its weight is zero)
-  auto request = [&](int i) {
-    const uint32_t bar = bars + 8u * (i % p.stages);
-    if (lane == 0) mbar_expect_tx(bar, uint32_t(kLdKeys * p.w * 2));
-    __syncwarp();
-    const uint32_t dst = smem_u32(ld_smem) + (i % p.stages) * tile_bytes;
-#pragma unroll
-    for (int k = 0; k < kLdKeys / 32; ++k) {
-      const int r = k * 32 + lane, pos = min(t0 + i * kLdKeys + r, t1 - 1);
-      const long long src = (long long)bt[pos / p.block_size] * p.block_size + pos % p.block_size;
-      ld_bulk(dst + r * pitch, p.cache + src * p.w, uint32_t(p.w * 2), bar);
-    }
-  };
-  if (warp == 0)
-    for (int i = 0; i < p.stages - 1 && i < tiles; ++i) request(i);
-
-  const int nch = p.c / 64;                      // 8-column blocks per warp in the value product (up to 8)
-  float o[MT][8][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int n = 0; n < 8; ++n)
-#pragma unroll
-      for (int r = 0; r < 4; ++r) o[m][n][r] = 0.f;
   const int g = lane >> 2, qd = lane & 3;
-  const int my_head = threadIdx.x / TPH, sub = threadIdx.x % TPH;
+  const int nch = FULL ? 8 : p.c / 64;           // 8-column blocks per warp in the value product (up to 8)
+  const int my_head = (threadIdx.x % kLdRole) / TPH, sub = threadIdx.x % TPH;
   float m_run = -INFINITY, l_run = 0.f;
-  const int kg = warp & 3, half = warp >> 2, ksteps = p.w / 32;       // per half
-  const uint32_t q_addr = smem_u32(q_s) + (lane & 15) * pitch + (lane >> 4) * 16 + half * (p.w / 2) * 2;
+  float o[MT][8][4];
   bool ok = true;
 
-  for (int i = 0; i < tiles; ++i) {
-    if (warp == 0 && i + p.stages - 1 < tiles) request(i + p.stages - 1);      // its stage was read in iteration i - 1
-    const uint32_t tile = smem_u32(ld_smem) + (i % p.stages) * tile_bytes;
-    const bool got = mbar_wait(bars + 8u * (i % p.stages), uint32_t(i / p.stages) & 1u, abort_flag, p.status, kStatusTimeoutFull);
-    if (got) {
-      float sc[MT][2][4];
+  if (warp < kLdRole / 32) {
+    // ------------------------------------------------------------------ scores and weights
+    const int kg = warp & 1, quarter = warp >> 1, nks = FULL ? kLdMaxKs : p.w / 64;
+    // A fragments of this warp's part of the query block: rows = heads (g and g + 8 of every block), zero past the last
+    uint32_t qa[MT][kLdMaxKs][4];
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+    for (int m = 0; m < MT; ++m) {
+      const bool lo_ok = m * 16 + g < heads, hi_ok = m * 16 + g + 8 < heads;
+      const __nv_bfloat16* q0 = p.q + ((long long)s * p.H + h0 + (lo_ok ? m * 16 + g : 0)) * p.w + quarter * (p.w / 4) + qd * 2;
+      const __nv_bfloat16* q1 = p.q + ((long long)s * p.H + h0 + (hi_ok ? m * 16 + g + 8 : 0)) * p.w + quarter * (p.w / 4) + qd * 2;
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int r = 0; r < 4; ++r) sc[m][n][r] = 0.f;
-      const uint32_t k_addr = tile + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16 + half * (p.w / 2) * 2;
-#pragma unroll 4
-      for (int ks = 0; ks < ksteps; ++ks) {
-        uint32_t b[4];
-        ld_ldsm_x4(k_addr + ks * 32, b);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t a[4];
-          ld_ldsm_x4(q_addr + m * 16 * pitch + ks * 32, a);
-          ld_mma(sc[m][0], a, b[0], b[1]);
-          ld_mma(sc[m][1], a, b[2], b[3]);
-        }
+      for (int ks = 0; ks < kLdMaxKs; ++ks) {
+        const bool in = ks < nks;
+        qa[m][ks][0] = in && lo_ok ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16) : 0u;
+        qa[m][ks][1] = in && hi_ok ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16) : 0u;
+        qa[m][ks][2] = in && lo_ok ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16 + 8) : 0u;
+        qa[m][ks][3] = in && hi_ok ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16 + 8) : 0u;
       }
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          float* dst = s_s + (half * MH + m * 16 + g) * kLdSPitch + kg * 16 + n * 8 + qd * 2;
-          *reinterpret_cast<float2*>(dst) = make_float2(sc[m][n][0], sc[m][n][1]);
-          *reinterpret_cast<float2*>(dst + 8 * kLdSPitch) = make_float2(sc[m][n][2], sc[m][n][3]);
-        }
     }
-    __syncthreads();
-    if (*abort_flag) { ok = false; break; }      // the same for all: the flag is written before the barrier or not at all
-    {
-      const float* s0 = s_s + my_head * kLdSPitch + sub * KPT;
-      const float* s1 = s0 + MH * kLdSPitch;
-      const int live = t1 - t0 - i * kLdKeys - sub * KPT;            // keys of this thread that exist
-      float v[KPT], mx = -INFINITY;
-#pragma unroll
-      for (int k = 0; k < KPT; k += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(s0 + k), b = *reinterpret_cast<const float4*>(s1 + k);
-        v[k] = (a.x + b.x) * p.scale_log2; v[k + 1] = (a.y + b.y) * p.scale_log2;
-        v[k + 2] = (a.z + b.z) * p.scale_log2; v[k + 3] = (a.w + b.w) * p.scale_log2;
-      }
-#pragma unroll
-      for (int k = 0; k < KPT; ++k) {
-        if (k >= live) v[k] = -INFINITY;
-        mx = fmaxf(mx, v[k]);
-      }
-#pragma unroll
-      for (int d = 1; d < TPH; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-      const float m_new = fmaxf(m_run, mx);      // finite: every tile has a key
-      const float f = exp2f(m_run - m_new);
-      float sum = 0.f;
-#pragma unroll
-      for (int k = 0; k < KPT; ++k) {
-        v[k] = exp2f(v[k] - m_new);
-        sum += v[k];
-      }
-#pragma unroll
-      for (int d = 1; d < TPH; d <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
-      l_run = l_run * f + sum;
-      m_run = m_new;
-      __nv_bfloat16* dst = p_s + my_head * kLdPPitch + sub * KPT;
-#pragma unroll
-      for (int k = 0; k < KPT; k += 4) stf4(dst + k, make_float4(v[k], v[k + 1], v[k + 2], v[k + 3]));
-      if (sub == 0) f_s[my_head] = f;
-    }
-    __syncthreads();
-    {
-      float f[MT][2];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) { f[m][0] = f_s[m * 16 + g]; f[m][1] = f_s[m * 16 + g + 8]; }
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int n = 0; n < 8; ++n) {
-          o[m][n][0] *= f[m][0]; o[m][n][1] *= f[m][0];
-          o[m][n][2] *= f[m][1]; o[m][n][3] *= f[m][1];
-        }
-      const uint32_t p_addr = smem_u32(p_s) + (lane & 15) * (kLdPPitch * 2) + (lane >> 4) * 16;
-      const uint32_t v_addr = tile + lane * pitch + warp * nch * 16;
-#pragma unroll
-      for (int kh = 0; kh < 2; ++kh) {           // 32 keys
-        uint32_t a[MT][2][4];
+    const int key = kg * 16 + (lane & 7) + ((lane >> 4) << 3), u0 = quarter * (p.w / 32) + ((lane >> 3) & 1);
+    const int key_at = unit_at(key, 0) & ~127;
+    int st = 0;
+    uint32_t phase = 0;
+    for (int i = 0; i < tiles; ++i) {
+      const int b = i & 1;
+      const uint32_t tile = smem_u32(ld_smem) + st * tile_bytes + key_at;
+      ok = ok && mbar_wait(full(st), phase, abort_flag, p.status, kStatusTimeoutFull);
+      if (++st == p.stages) { st = 0; phase ^= 1u; }
+      if (__all_sync(0xffffffffu, ok)) {
+        float sc[MT][2][4];
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
-          for (int k = 0; k < 2; ++k) ld_ldsm_x4(p_addr + m * 16 * (kLdPPitch * 2) + (kh * 2 + k) * 32, a[m][k]);
+          for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int n = 0; n < 8; ++n) {
-          if (n < nch) {
-            uint32_t b[4];
-            ld_ldsm_x4_trans(v_addr + kh * 32 * pitch + n * 16, b);
+            for (int r = 0; r < 4; ++r) sc[m][n][r] = 0.f;
+#pragma unroll
+        for (int ks = 0; ks < kLdMaxKs; ++ks) {
+          if (ks < nks) {
+            uint32_t kb[4];
+            const int u = u0 + ks * 2;            // 16-byte unit of the row
+            ld_ldsm_x4(tile + ((u >> 3) << (run_log + 7)) + (((u & 7) ^ (key & 7)) << 4), kb);
 #pragma unroll
             for (int m = 0; m < MT; ++m) {
-              ld_mma(o[m][n], a[m][0], b[0], b[1]);
-              ld_mma(o[m][n], a[m][1], b[2], b[3]);
+              ld_mma(sc[m][0], qa[m][ks], kb[0], kb[1]);
+              ld_mma(sc[m][1], qa[m][ks], kb[2], kb[3]);
             }
           }
         }
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            float* dst = s_s + ((b * 4 + quarter) * MH + m * 16 + g) * kLdSPitch + kg * 16 + n * 8 + qd * 2;
+            *reinterpret_cast<float2*>(dst) = make_float2(sc[m][n][0], sc[m][n][1]);
+            *reinterpret_cast<float2*>(dst + 8 * kLdSPitch) = make_float2(sc[m][n][2], sc[m][n][3]);
+          }
       }
+      // the quarters are there; a wait that ran out in one warp ends the loop in all
+      if (!ld_bar_and(ok)) { ok = false; break; }
+      const float* sr = s_s + (b * 4 * MH + my_head) * kLdSPitch + sub * KPT;
+      const int first = t0 + i * kLdKeys + sub * KPT;                // this thread's keys that are visible: in [lo, t1)
+      float v[KPT], mx = -INFINITY;
+#pragma unroll
+      for (int k = 0; k < KPT; ++k) v[k] = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if constexpr (KPT == 4) {
+          const float4 a = *reinterpret_cast<const float4*>(sr + j * MH * kLdSPitch);
+          v[0] += a.x; v[1] += a.y; v[2] += a.z; v[3] += a.w;
+        } else {
+          const float2 a = *reinterpret_cast<const float2*>(sr + j * MH * kLdSPitch);
+          v[0] += a.x; v[1] += a.y;
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < KPT; ++k) {
+        v[k] = first + k < t1 && first + k >= lo ? v[k] * p.scale_log2 : -INFINITY;
+        mx = fmaxf(mx, v[k]);
+      }
+      // The reference the exponents are taken from moves only when a score passes it by more than 2^8 (and for the first tile).
+      const bool over = mx > m_run + 8.f;
+      float f = 1.f;
+      if (__any_sync(0xffffffffu, over)) {
+#pragma unroll
+        for (int d = 1; d < TPH; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+        if (mx > m_run + 8.f) {
+          f = exp2f(m_run - mx);                 // zero for the first tile
+          l_run *= f;
+          m_run = mx;
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < KPT; ++k) {
+        v[k] = exp2f(v[k] - m_run);
+        l_run += v[k];                           // this thread's share of the sum
+      }
+      if (i >= 2) ok = mbar_wait(p_free(b), uint32_t((i >> 1) - 1) & 1u, abort_flag, p.status, kStatusTimeoutEmpty);
+      __nv_bfloat16* dst = p_s + (b * MH + my_head) * kLdPPitch + sub * KPT;
+      if constexpr (KPT == 4) stf4(dst, make_float4(v[0], v[1], v[2], v[3]));
+      else stf2(dst, make_float2(v[0], v[1]));
+      if (sub == 0) f_s[b * MH + my_head] = f;
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_full(b));
     }
-    __syncthreads();                             // the stage, the scores and the weights may be written again
-  }
-  if (!ok) {
-    // a copy never arrived: the other requested stages get one more bounded wait each before the CTA leaves
-    if (warp == 0)
-      for (int st = 0; st < p.stages; ++st) {
-        mbar_wait(bars + 8u * st, 0u, &drain_s, p.status, kStatusTimeoutFull);
-        mbar_wait(bars + 8u * st, 1u, &drain_s, p.status, kStatusTimeoutFull);
+  } else {
+    // ------------------------------------------------------------------ values, and the copies (first warp of these)
+    const int pw = warp - kLdRole / 32;
+    const int* bt = p.tables + (long long)s * p.max_blocks;
+    // Lane l brings the l-th run of rows of every tile: the block of the table it lies in, and where in the block.
+    int blk = (t0 + lane * run) / p.block_size, in_blk = (t0 + lane * run) % p.block_size, asked = 0, ask_st = 0;
+    auto next_row = [&]() {                      // its first row of the next tile in the cache (-1: none), then one tile on
+      const int row = lane < kLdKeys >> run_log && t0 + asked * kLdKeys + lane * run < t1 ? bt[blk] * p.block_size + in_blk : -1;
+      if (run < kLdKeys) blk += kLdKeys >> run_log;
+      else if ((in_blk += kLdKeys) == p.block_size) { in_blk = 0; ++blk; }
+      return row;
+    };
+    auto request = [&](int row) {                // pages are allocated whole: runs come whole
+      const int rows = min(kLdKeys, ((t1 - t0 - asked * kLdKeys + run - 1) >> run_log) << run_log);
+      if (lane == 0) mbar_expect_tx(full(ask_st), uint32_t(rows * p.w * 2));
+      __syncwarp();
+      if (row >= 0) tma_load_3d(smem_u32(ld_smem) + ask_st * tile_bytes + lane * run_bytes, &tmap, full(ask_st), 0, row, 0);
+      ++asked;
+      if (++ask_st == p.stages) ask_st = 0;
+    };
+    int row = -1;                                // of the next tile to ask for
+    if (pw == 0) {
+      for (int i = 0; i < p.stages - 1 && i < tiles; ++i) request(next_row());
+      row = next_row();
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int r = 0; r < 4; ++r) o[m][n][r] = 0.f;
+    const int lane_at = unit_at(lane, 0) & ~127;
+    int st = 0, old_st = 0;
+    uint32_t phase = 0, old_phase = 0;
+    for (int i = 0; i < tiles; ++i) {
+      const int b = i & 1;
+      if (pw == 0 && asked < tiles) {                          // into the stage of tile i - 1
+        if (i > 0) ok = mbar_wait(empty(old_st), old_phase, abort_flag, p.status, kStatusTimeoutEmpty);
+        if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+        request(row);
+        row = next_row();                                      // on its way until the next request
       }
-    return;
+      ok = mbar_wait(full(st), phase, abort_flag, p.status, kStatusTimeoutFull) &&
+           mbar_wait(p_full(b), uint32_t(i >> 1) & 1u, abort_flag, p.status, kStatusTimeoutFull);
+      if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+      const int tail = t1 - t0 - i * kLdKeys;
+      if (tail < kLdKeys) {
+        // rows past the last key may hold anything: zeros where this warp reads, so that zero weights do not meet a NaN
+        if (lane >= tail)
+          for (int n = 0; n < nch; ++n)
+            *reinterpret_cast<uint4*>(ld_smem + st * tile_bytes + unit_at(lane, pw * nch + n)) = make_uint4(0u, 0u, 0u, 0u);
+        __syncwarp();
+      }
+      bool same = true;
+      float f[MT][2];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        f[m][0] = f_s[b * MH + m * 16 + g];
+        f[m][1] = f_s[b * MH + m * 16 + g + 8];
+        same = same && f[m][0] == 1.f && f[m][1] == 1.f;
+      }
+      if (!__all_sync(0xffffffffu, same)) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int n = 0; n < 8; ++n) {
+            o[m][n][0] *= f[m][0]; o[m][n][1] *= f[m][0];
+            o[m][n][2] *= f[m][1]; o[m][n][3] *= f[m][1];
+          }
+      }
+      const uint32_t tile = smem_u32(ld_smem) + st * tile_bytes + lane_at;
+      const uint32_t p_addr = smem_u32(p_s) + b * MH * kLdPPitch * 2 + (lane & 15) * (kLdPPitch * 2) + (lane >> 4) * 16;
+      uint32_t a[MT][2][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int k = 0; k < 2; ++k) ld_ldsm_x4(p_addr + m * 16 * (kLdPPitch * 2) + k * 32, a[m][k]);
+#pragma unroll
+      for (int n = 0; n < 8; n += 2) {           // two column blocks at a time: four products between dependent ones
+        if (n < nch) {
+          uint32_t vb[2][4];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int u = pw * nch + n + e;
+            if (n + e < nch) ld_ldsm_x4_trans(tile + ((u >> 3) << (run_log + 7)) + (((u & 7) ^ (lane & 7)) << 4), vb[e]);
+          }
+#pragma unroll
+          for (int k = 0; k < 2; ++k)
+#pragma unroll
+            for (int e = 0; e < 2; ++e)
+#pragma unroll
+              for (int m = 0; m < MT; ++m)
+                if (n + e < nch) ld_mma(o[m][n + e], a[m][k], vb[e][2 * k], vb[e][2 * k + 1]);
+        }
+      }
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(p_free(b)); mbar_arrive(empty(st)); }
+      old_st = st;
+      old_phase = phase;
+      if (++st == p.stages) { st = 0; phase ^= 1u; }
+    }
   }
-  if (sub == 0) { m_s[my_head] = m_run; l_s[my_head] = l_run; }
+  if (*abort_flag && warp == 0) {
+    // a copy never arrived: the other requested stages get one more bounded wait each before the CTA goes on
+    for (int st = 0; st < p.stages; ++st) {
+      mbar_wait(full(st), 0u, &drain_s, p.status, kStatusTimeoutFull);
+      mbar_wait(full(st), 1u, &drain_s, p.status, kStatusTimeoutFull);
+    }
+  }
+#pragma unroll
+  for (int d = 1; d < TPH; d <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, d);
+  const bool maker = warp >= kLdRole / 32;       // holds outputs; the others hold maxima and sums
+  const int pw = maker ? warp - kLdRole / 32 : 0;
+  if (!maker && sub == 0) {
+    m_s[my_head] = ok ? m_run : -INFINITY;
+    l_s[my_head] = ok ? l_run : 0.f;
+  }
   __syncthreads();
   if (p.splits > 1 && threadIdx.x < heads) {
     float* st = p.stat + (((long long)s * p.H + h0 + threadIdx.x) * p.splits + sp) * 2;
     st[0] = m_s[threadIdx.x];
     st[1] = l_s[threadIdx.x];
   }
+  if (tiles == 0 || !maker) return;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -364,7 +450,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
       for (int n = 0; n < 8; ++n) {
         if (n < nch) {
-          const int col = (warp * nch + n) * 8 + qd * 2;
+          const int col = (pw * nch + n) * 8 + qd * 2;
           const float2 v = make_float2(o[m][n][e * 2], o[m][n][e * 2 + 1]);
           if (p.splits > 1) stf2(p.part + (row * p.splits + sp) * p.c + col, v);
           else stf2(p.out + row * p.c + col, make_float2(v.x * inv, v.y * inv));
@@ -373,38 +459,57 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     }
 }
 
-// out[row, :] from the splits of one (sequence, head).
+// out[row, :] from the splits of one (sequence, head): a thread per four columns, eight splits in flight.
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part, const float* __restrict__ stat,
                                                            __nv_bfloat16* __restrict__ out, int splits, int c) {
+  __shared__ float share[kLdMaxSplits];
   const long long row = blockIdx.x;
   const float2* st = reinterpret_cast<const float2*>(stat) + row * splits;
-  float m = -INFINITY, l = 0.f;
-  for (int i = 0; i < splits; ++i) m = fmaxf(m, st[i].x);
-  for (int i = 0; i < splits; ++i) l += st[i].y > 0.f ? st[i].y * exp2f(st[i].x - m) : 0.f;
-  const float inv = 1.f / l;
-  for (int col = threadIdx.x * 4; col < c; col += 128 * 4) {
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int i = 0; i < splits; ++i) {
-      if (st[i].y > 0.f) {                       // a split without keys has written no outputs
-        const float f = exp2f(st[i].x - m);
-        const float4 v = ldf4(part + (row * splits + i) * c + col);
-        a.x = fmaf(f, v.x, a.x); a.y = fmaf(f, v.y, a.y); a.z = fmaf(f, v.z, a.z); a.w = fmaf(f, v.w, a.w);
-      }
+  if (threadIdx.x < 32) {
+    float m = -INFINITY, l = 0.f;
+    for (int i = threadIdx.x; i < splits; i += 32) m = fmaxf(m, st[i].x);
+    m = warp_max(m);
+    for (int i = threadIdx.x; i < splits; i += 32) {
+      const float2 v = st[i];
+      const float f = v.y > 0.f ? exp2f(v.x - m) : 0.f;
+      share[i] = f;
+      l = fmaf(v.y, f, l);
     }
-    stf4(out + row * c + col, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
+    l = warp_sum(l);
+    for (int i = threadIdx.x; i < splits; i += 32) share[i] /= l;
+  }
+  __syncthreads();
+  for (int col = threadIdx.x * 4; col < c; col += 128 * 4) {
+    const float* src = part + row * splits * c + col;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i0 = 0; i0 < splits; i0 += 8) {
+      float4 v[8];
+      float f[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        f[i] = i0 + i < splits ? share[i0 + i] : 0.f;
+        if (f[i] > 0.f) v[i] = ldf4(src + (long long)(i0 + i) * c);    // a split without keys has written no outputs
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (f[i] > 0.f) {
+          a.x = fmaf(f[i], v[i].x, a.x); a.y = fmaf(f[i], v[i].y, a.y); a.z = fmaf(f[i], v[i].z, a.z); a.w = fmaf(f[i], v[i].w, a.w);
+        }
+    }
+    stf4(out + row * c + col, a);
   }
 }
 
-template <int MT>
-static int launch_latent_decode(LatentDecodeParams& p, int S, cudaStream_t st) {
+template <int MT, bool FULL>
+static int launch_latent_decode(const CUtensorMap& tmap, LatentDecodeParams& p, int S, cudaStream_t st) {
   constexpr int MH = MT * 16;
   p.stages = kLdMaxStages;
   while (p.stages > 2 && ld_smem_bytes(p.w, MH, p.stages) > 227 * 1024) --p.stages;
   const int smem = ld_smem_bytes(p.w, MH, p.stages);
   if (smem > 227 * 1024) return -4;
-  auto kern = latent_decode_kernel<MT>;
+  auto kern = latent_decode_kernel<MT, FULL>;
   LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  kern<<<dim3(p.splits, (p.H + MH - 1) / MH, S), kLdThreads, smem, st>>>(p);
+  kern<<<dim3(p.splits, (p.H + MH - 1) / MH, S), kLdThreads, smem, st>>>(tmap, p);
   LT_LAUNCH_CHECK();
   return 0;
 }
@@ -433,19 +538,26 @@ int lt_latent_rope(int fp32, void* proj, long long ld, int n, int H, int d, int 
 }
 
 // out [S, H, c] = attention of q [S, H, w] over the rows of each sequence's pages (the newest `window`, 0: all); c and w multiples
-// of 64, c <= 512.  part [S * H, splits, c] and stat [S * H, splits, 2] are scratch (unused with one split).
+// of 64, c <= 512, w <= 576; block_size 8, 16 or a multiple of 32; the cache has num_blocks blocks.  part [S * H, splits, c] and stat [S * H, splits, 2] are scratch (unused with one split).
+// splits <= 64.
 int lt_latent_decode(const void* q, const void* cache, const int* tables, const int* ctx, float* part, float* stat, void* out, int S,
-                     int H, int c, int w, int block_size, int max_blocks, int splits, int window, float scale, void* stream) {
+                     int H, int c, int w, int num_blocks, int block_size, int max_blocks, int splits, int window, float scale, void* stream) {
   using namespace lt;
   if (S == 0) return 0;
-  if (H < 1 || c < 64 || c > 512 || (c & 63) || (w & 63) || w < c || w > 1024 || splits < 1 || splits > 65535 || S > 65535 ||
-      (splits > 1 && (!part || !stat)) || (reinterpret_cast<uintptr_t>(cache) & 15) || (reinterpret_cast<uintptr_t>(q) & 15))
+  if (H < 1 || c < 64 || c > 512 || (c & 63) || (w & 63) || w < c || w > 64 * kLdMaxKs || splits < 1 || splits > kLdMaxSplits || S > 65535 ||
+      (block_size != 8 && block_size != 16 && block_size % 32 != 0) || num_blocks < 1 || (splits > 1 && (!part || !stat)) || (reinterpret_cast<uintptr_t>(cache) & 15) || (reinterpret_cast<uintptr_t>(q) & 15))
     return -4;
-  LatentDecodeParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache), tables, ctx, part, stat,
+  LatentDecodeParams p{static_cast<const __nv_bfloat16*>(q), tables, ctx, part, stat,
                        static_cast<__nv_bfloat16*>(out), H, c, w, block_size, max_blocks, splits, window, 0,
                        scale * 1.4426950408889634f, device_status_word()};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int rc = H <= 16 ? launch_latent_decode<1>(p, S, st) : launch_latent_decode<2>(p, S, st);
+  CUtensorMap tmap;
+  const int r = encode_tmap_3d(&tmap, cache, 2, 64, (uint64_t)num_blocks * block_size, w / 64, (uint64_t)w * 2, 128, 64,
+                               block_size < kLdKeys ? block_size : kLdKeys, w / 64, 1);
+  if (r) return 1000 + r;
+  const bool full = c == 512 && w == 64 * kLdMaxKs;
+  const int rc = H <= 16 ? (full ? launch_latent_decode<1, true>(tmap, p, S, st) : launch_latent_decode<1, false>(tmap, p, S, st))
+                         : (full ? launch_latent_decode<2, true>(tmap, p, S, st) : launch_latent_decode<2, false>(tmap, p, S, st));
   if (rc != 0 || splits == 1) return rc;
   latent_merge_kernel<<<S * H, 128, 0, st>>>(part, stat, static_cast<__nv_bfloat16*>(out), splits, c);
   LT_LAUNCH_CHECK();

@@ -193,7 +193,7 @@ int lt_latent_rope(int fp32, void* proj, long long ld, int n, int H, int d, int 
                    const float* c_norm, float eps, const int* positions, const int* slots, const double* freq, float gain, void* q_out,
                    int q_ld, int q_col, void* cache, void* lin, void* stream);
 int lt_latent_decode(const void* q, const void* cache, const int* tables, const int* ctx, float* part, float* stat, void* out, int S,
-                     int H, int c, int w, int block_size, int max_blocks, int splits, int window, float scale, void* stream);
+                     int H, int c, int w, int num_blocks, int block_size, int max_blocks, int splits, int window, float scale, void* stream);
 int lt_moe_plan(const float* logits, const float* correction, float* weight, int* slot, int* src, int* group, int* group_rows, int* live,
                 void* pairs, int* counts, const void* x, void* xs, int row_bytes, int N, int E, int top, int block_rows, void* stream);
 int lt_moe_grouped_gemm(const void* A, const void* W, void* C, const int* group, const int* live, int max_blocks, int experts, int N,

@@ -18,7 +18,7 @@ _vp, _i, _ll, _f = c_void_p, c_int, c_longlong, c_float
 _SIGS = {
     "lt_residual_norm": [_i, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _i, _vp, _f, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
     "lt_latent_rope": [_i, _vp, _ll] + [_i] * 8 + [_vp, _f, _vp, _vp, _vp, _f, _vp, _i, _i, _vp, _vp, _vp],
-    "lt_latent_decode": [_vp] * 7 + [_i] * 8 + [_f, _vp],
+    "lt_latent_decode": [_vp] * 7 + [_i] * 9 + [_f, _vp],
     "lt_flash_fwd_shared": [_vp] * 6 + [_i] * 5 + [_ll] * 4 + [_f, _i, _vp],
     "lt_moe_plan": [_vp] * 12 + [_i] * 5 + [_vp],
     "lt_moe_grouped_gemm": [_vp] * 5 + [_i] * 4 + [_vp],
@@ -121,7 +121,7 @@ _SIGS = {
 _bound = {}
 
 # Kernels launched per native call; `launch_count()` is what bench.py reports as "gpu_launches".
-_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_paged_decode_window": 2, "lt_latent_decode": 2, "lt_mlstm_prefill": 4, "lt_rglru_scan": 3, "lt_rglru_step": 2, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
+_LAUNCHES_PER_CALL = {"lt_gemm_num_tiles": 0, "lt_gemm_skinny_set_target": 0, "lt_adam_q8": 3, "lt_set_wait_budget_cycles": 0, "lt_norm_bwd": 2, "lt_paged_decode": 2, "lt_paged_decode_window": 2, "lt_mlstm_prefill": 4, "lt_rglru_scan": 3, "lt_rglru_step": 2, "lt_flash_bwd": 3, "lt_status_fetch": 0, "lt_sm_count": 0, "lt_gemm_set_tail_split": 0, "lt_reduce_parts": 0, "lt_reduce_all": 2, "lt_gemm_set_pair_mode": 0, "lt_flash_bwd_set_trace": 0, "lt_flash_fwd_set_trace": 0, "lt_norm_bwd_ctas": 0,
                       "lt_adam_chunk_elems": 0}
 _launches = [0]
 
@@ -1092,16 +1092,11 @@ def shared_rope_fwd(q, k, k_rot, v, *, scale: float, window: int = 0):
 
 
 def latent_splits(S: int, H: int, keys: int, sms: int = 148) -> int:
-    """Splits of the key range per sequence: as few rounds of tiles over the SMs (one CTA each) as possible; a split costs about
-    two tiles on top of its own."""
+    """Splits of the key range per sequence: the rounds over the SMs (one CTA each) times the 32-key tiles of a split, a CTA costing
+    about eight tiles beside them and a split a twentieth of one in the merge."""
     ctas = S * ((H + 31) // 32)
-    best, cost = 1, None
-    for n in range(1, max(1, min(64, (keys + 63) // 64)) + 1):
-        waves = (ctas * n + sms - 1) // sms
-        c = waves * ((keys + 64 * n - 1) // (64 * n) + 2) + (2 if n > 1 else 0)
-        if cost is None or c < cost:
-            best, cost = n, c
-    return best
+    cost = lambda n: (ctas * n + sms - 1) // sms * ((keys + 32 * n - 1) // (32 * n) + 8) + 0.05 * n
+    return min(range(1, max(1, min(64, (keys + 31) // 32)) + 1), key=cost)
 
 
 def latent_decode(q, cache, tables, ctx, *, rank: int, window: int, scale: float, max_keys: int, splits: int = 0):
@@ -1113,7 +1108,7 @@ def latent_decode(q, cache, tables, ctx, *, rank: int, window: int, scale: float
     o = torch.empty((S, H, rank), dtype=q.dtype, device=q.device)
     part = torch.empty(S * H * splits * (rank + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
     rc = _fn("lt_latent_decode")(q.data_ptr(), cache.data_ptr(), tables.data_ptr(), ctx.data_ptr(), _p(part),
-                                 part[S * H * splits * rank:].data_ptr() if splits > 1 else None, o.data_ptr(), S, H, rank, w, cache.shape[2],
+                                 part[S * H * splits * rank:].data_ptr() if splits > 1 else None, o.data_ptr(), S, H, rank, w, cache.shape[0], cache.shape[2],
                                  tables.shape[1], splits, int(window), float(scale), _stream())
     _check(rc, "lt_latent_decode")
     return o

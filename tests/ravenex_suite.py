@@ -67,7 +67,7 @@ def weights(cfg, seed=0):
     gen = torch.Generator().manual_seed(seed)
     w = {n: random_tensor(n, s, gen) for n, s in tensor_shapes(RavenexConfig.parse(cfg)).items()}
     for n in w:
-        f = 3.0 if n.endswith("mix.q") else 2.0 if n.endswith(("router", "correction")) else 0
+        f = 2.0 if n.endswith("mix.q") else 2.0 if n.endswith(("router", "correction")) else 0
         if f:
             w[n] = (w[n].float() * f).to(torch.bfloat16)
     return w
