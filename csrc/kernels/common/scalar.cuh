@@ -93,6 +93,8 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
 }
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// SiLU for results that leave as bf16: the quick exponential and quotient (a few units in the last place of fp32).
+__device__ __forceinline__ float silu_quick_f(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 __device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));

@@ -232,8 +232,8 @@ gemm_skinny_kernel(const SkinnyParams p) {
         float v0 = acc[m][f][h * 2], v1 = acc[m][f][h * 2 + 1];
         if constexpr (GLU) {
           const float u0 = acc[m][f + 2][h * 2], u1 = acc[m][f + 2][h * 2 + 1];
-          v0 = (p.act == 1 ? gelu_tanh_f(v0) : v0 * sigmoid_f(v0)) * u0;
-          v1 = (p.act == 1 ? gelu_tanh_f(v1) : v1 * sigmoid_f(v1)) * u1;
+          v0 = (p.act == 1 ? gelu_tanh_f(v0) : silu_quick_f(v0)) * u0;
+          v1 = (p.act == 1 ? gelu_tanh_f(v1) : silu_quick_f(v1)) * u1;
         } else if (p.residual) {
           const float2 rv = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p.residual + (long long)row * p.ldr + col));
           v0 += rv.x;

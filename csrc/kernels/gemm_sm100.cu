@@ -52,6 +52,27 @@ static int launch_gemm_pair(const CUtensorMap& tmA, const CUtensorMap& tmB, cons
   return 0;
 }
 
+template <int BLOCK_N, int EPI>
+__global__ void __launch_bounds__(kGemmThreads, 1)
+gemm_staged_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const __grid_constant__ CUtensorMap tmC,
+                   const GemmParams p) {
+  gemm_body<BLOCK_N, 0, 0, 0, false, EPI>(&tmA, &tmB, p, NoGate(), NoDone(), 0, &tmC);
+}
+
+template <int BLOCK_N, int EPI>
+static int launch_staged(const CUtensorMap& tmA, const CUtensorMap& tmB, const CUtensorMap& tmC, const GemmParams& p, int grid,
+                         cudaStream_t st) {
+  static bool configured = false;
+  auto kern = gemm_staged_kernel<BLOCK_N, EPI>;
+  if (!configured) {
+    LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, GemmCfg<BLOCK_N>::kStagedSmemBytes));
+    configured = true;
+  }
+  kern<<<grid, kGemmThreads, GemmCfg<BLOCK_N>::kStagedSmemBytes, st>>>(tmA, tmB, tmC, p);
+  LT_LAUNCH_CHECK();
+  return 0;
+}
+
 template <int BLOCK_N>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_block_diag_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const GemmParams p) {
@@ -184,6 +205,35 @@ int lt_gemm_e4m3(const void* A, const void* B, void* C, int M, int N, int K, lon
   // e4m3 rows seen as rows of 2-byte units of half the extent (the copy is byte-identical)
   return gemm_launch(4, A, B, C, M, N, K / 2, lda / 2, ldb / 2, ldc, 0, 0, out_fp32, bias, residual, ldr, act, 0, alpha, 0, 0, stream,
                      a_scale, b_scale);
+}
+
+// C [M, N] bf16 = alpha * A [M, K] @ B [N, K]^T with the staged epilogue; block_n 0: choose, 128 or 256.  With act (1 GELU, 2 SiLU): B is
+// [2 N, K], gate rows, then up rows, and C = act(gate) * up.  Pitches in elements, multiples of 8; N a multiple of 8.
+int lt_gemm_staged(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb, long long ldc, int act,
+                   float alpha, int block_n, void* stream) {
+  using namespace lt;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((lda & 7) || (ldb & 7) || (ldc & 7) || (N & 7) || act < 0 || act > 2 || (reinterpret_cast<uintptr_t>(A) & 15) ||
+      (reinterpret_cast<uintptr_t>(B) & 15) || (reinterpret_cast<uintptr_t>(C) & 15))
+    return -int(kStatusBadArgument);
+  const int sms = sm_count();
+  if (act) block_n = 256;
+  else if (block_n != 128 && block_n != 256) block_n = pick_block_n(M, N, sms);
+  GemmParams p{};
+  p.M = M; p.N = N; p.K = K;
+  p.C = C; p.ldc = ldc; p.alpha = alpha;
+  p.glu_act = act;
+  p.status = device_status_word();
+  fill_tiles(p, act ? 128 : block_n);
+  CUtensorMap tmA, tmB, tmC;
+  int r = make_operand_maps(&tmA, &tmB, A, B, M, act ? 2 * N : N, K, lda, ldb, 0, 0, act ? 128 : block_n);
+  if (r) return r;
+  r = make_staged_map(&tmC, C, M, N, ldc);
+  if (r) return 3000 + r;
+  const int grid = p.num_tiles < sms ? p.num_tiles : sms;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (act) return launch_staged<256, kEpiGlu>(tmA, tmB, tmC, p, grid, st);
+  return block_n == 256 ? launch_staged<256, kEpiStaged>(tmA, tmB, tmC, p, grid, st) : launch_staged<128, kEpiStaged>(tmA, tmB, tmC, p, grid, st);
 }
 
 // C[M, blocks * nb] (fp32) = A[M, blocks * K] @ blockdiag(B_0 .. )^T with B [blocks, nb, K]: columns z * nb .. of C are the

@@ -19,6 +19,7 @@
 #pragma once
 #include "common/host.h"
 #include "common/ptx.cuh"
+#include "common/scalar.cuh"
 
 namespace lt {
 
@@ -78,6 +79,8 @@ struct GemmParams {
   // times b_scale[c] (fp32, nullptr: 1).
   const float* a_scale;
   const float* b_scale;
+  // Gated epilogue (kEpiGlu): 1 GELU (tanh form), 2 SiLU; B holds N gate rows, then N up rows (per group, with group_of_mblk).
+  int glu_act;
   // Block-diagonal B (one-CTA kernel, both operands K-major): columns come in groups of diag_n, and group z multiplies the K
   // columns of A that start at z * K.  A's tensor map spans all groups; a K tile that runs past K meets zeros of B.  0: off.
   int diag_n;
@@ -116,7 +119,14 @@ struct GemmCfg {
   static constexpr int kTmemCols = 2 * BLOCK_N;
   static constexpr int kBarrierBytes = 512;
   static constexpr int kSmemBytes = kStages * kStageBytes + 1024 + kBarrierBytes;
+  // With a staged epilogue: two 32 x 64 bf16 pieces for each of the four epilogue warps behind the barriers.
+  static constexpr int kOffStaging = kStages * kStageBytes + 1024;
+  static constexpr int kStagedSmemBytes = kOffStaging + 4 * 2 * 4096 + 1024;
 };
+
+// Epilogues of the one-CTA kernel: everything in registers and stored from there; bf16 results staged in shared memory and
+// written by TMA (alpha alone is applied); the same with act(gate) * up of a tile's two column halves.
+enum { kEpiDirect = 0, kEpiStaged = 1, kEpiGlu = 2 };
 
 struct NoGate {
   __device__ __forceinline__ bool operator()(int, int, int, int*) const { return true; }
@@ -324,10 +334,13 @@ __device__ __forceinline__ void store_f32_lines(const GemmParams& p, int row, in
 // format bits of the run-time instruction descriptor), 2 = kind::tf32, 3 = kind::i8, 4 = kind::f8f6f4 with e4m3 operands.  It is a template parameter and
 // not a run-time branch on purpose: a kernel that contains tcgen05.mma instructions of more than one kind ran its
 // bf16 MMAs at half rate (measured: 1000 instead of 512 cycles per 256 x 256 x 64 block with no loads in flight).
+// EPI: see above; staged epilogues take the output's tensor map (box 64 columns x 32 rows, 128-byte swizzle), and with kEpiGlu a
+// tile is BLOCK_N / 2 result columns, tmB's box BLOCK_N / 2 rows.
 // DIAG: the block-diagonal product (GemmParams::diag_n) with fp32 results and nothing else in the epilogue.
-template <int BLOCK_N, int A_MAJOR, int B_MAJOR, int MMA_KIND = 0, bool DIAG = false, class TileGate, class TileDone>
+template <int BLOCK_N, int A_MAJOR, int B_MAJOR, int MMA_KIND = 0, bool DIAG = false, int EPI = kEpiDirect, class TileGate, class TileDone>
 __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensorMap* tmB, const GemmParams& p,
-                                          TileGate gate, TileDone done, int cta_first = 0) {
+                                          TileGate gate, TileDone done, int cta_first = 0, const CUtensorMap* tmC = nullptr) {
+  static_assert(EPI == kEpiDirect || (B_MAJOR == 0 && !DIAG), "staged epilogues go with K-major weights");
   // CTAs [0, cta_first) of the grid belong to another role of a fused kernel; the GEMM uses the rest.
   const int cta_id = int(blockIdx.x) - cta_first;
   const int cta_count = int(gridDim.x) - cta_first;
@@ -403,7 +416,10 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensor
               tma_load_2d(a_dst + i * (64 * kBlockK * 2), tmA, fb, m_blk * kBlockM + i * 64, kb * kBlockK);
           }
           const int b_off = p.group_of_mblk ? p.group_of_mblk[m_blk] * p.b_group_rows : 0;
-          if (B_MAJOR == 0) {
+          if constexpr (EPI == kEpiGlu) {
+            tma_load_2d(b_dst, tmB, fb, kb * kBlockK, b_off + n_blk * (BLOCK_N / 2));
+            tma_load_2d(b_dst + Cfg::kBBytes / 2, tmB, fb, kb * kBlockK, b_off + p.N + n_blk * (BLOCK_N / 2));
+          } else if (B_MAJOR == 0) {
             tma_load_2d(b_dst, tmB, fb, kb * kBlockK, b_off + n_blk * BLOCK_N);
           } else {
 #pragma unroll
@@ -456,6 +472,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensor
     // ------------------------------------------------------------------ epilogue (4 warps)
     const int quarter = warp & 3;  // TMEM lane quarter this warp may read
     WorkItem w;
+    [[maybe_unused]] int staged = 0;   // pieces this warp has handed to TMA
     for (int it = 0; get_item(p, cta_id, cta_count, it, w); ++it) {
       int m_blk, n_blk;
       tile_coords(p, w.tile, m_blk, n_blk);
@@ -466,6 +483,53 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensor
       tc_fence_after();
       const int row = m_blk * kBlockM + quarter * 32 + lane;
       const uint32_t t_addr = tmem_base + (uint32_t(quarter * 32) << 16) + buf * BLOCK_N;
+      if constexpr (EPI != kEpiDirect) {
+        constexpr int OUT_N = EPI == kEpiGlu ? BLOCK_N / 2 : BLOCK_N;
+#pragma unroll 1
+        for (int c = 0; c < OUT_N / 64; ++c) {
+          if (n_blk * OUT_N + c * 64 >= p.N) break;
+          uint32_t w[32];                          // 64 results of this lane's row as bf16 pairs
+#pragma unroll
+          for (int hh = 0; hh < 2; ++hh) {
+            uint32_t r[32];
+            tmem_ld_32x32(t_addr + c * 64 + hh * 32, r);
+            if constexpr (EPI == kEpiGlu) {
+              uint32_t u[32];
+              tmem_ld_32x32(t_addr + OUT_N + c * 64 + hh * 32, u);
+              tmem_ld_wait();
+#pragma unroll
+              for (int j = 0; j < 32; ++j) {
+                const float g = __uint_as_float(r[j]) * p.alpha;
+                r[j] = __float_as_uint((p.glu_act == 1 ? gelu_tanh_f(g) : silu_quick_f(g)) * (__uint_as_float(u[j]) * p.alpha));
+              }
+            } else {
+              tmem_ld_wait();
+#pragma unroll
+              for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * p.alpha);
+            }
+#pragma unroll
+            for (int j = 0; j < 16; ++j) w[hh * 16 + j] = pack_bf16x2(__uint_as_float(r[2 * j]), __uint_as_float(r[2 * j + 1]));
+          }
+          uint8_t* piece = smem + Cfg::kOffStaging + ((warp - 2) * 2 + (staged & 1)) * 4096;
+          if (lane == 0) tma_store_wait_read<1>();   // the store that last used this piece has read it
+          __syncwarp();
+#pragma unroll
+          for (int u = 0; u < 8; ++u)
+            *reinterpret_cast<uint4*>(piece + lane * 128 + ((u ^ (lane & 7)) << 4)) = make_uint4(w[u * 4], w[u * 4 + 1], w[u * 4 + 2], w[u * 4 + 3]);
+          fence_proxy_async();
+          __syncwarp();
+          if (lane == 0) {
+            if (m_blk * kBlockM + quarter * 32 < p.M)
+              tma_store_2d(tmC, smem_u32(piece), n_blk * OUT_N + c * 64, m_blk * kBlockM + quarter * 32);
+            tma_store_commit();
+          }
+          ++staged;
+        }
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(tempty_bar(buf));
+        continue;
+      }
       if (w.split > 0) {
         // contributor of a split tile: raw accumulators to the workspace, then one arrival per warp
         float* ws = p.sk_ws + ((long long)(w.slot * (p.sk_split - 1) + (w.split - 1)) * (BLOCK_N / 32)) * (kBlockM * 32) +
@@ -546,6 +610,9 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA, const CUtensor
         done(m_blk, n_blk);
       }
     }
+    if constexpr (EPI != kEpiDirect) {
+      if (lane == 0) tma_store_wait<0>();
+    }
   }
 
   // ------------------------------------------------------------------ teardown
@@ -621,6 +688,11 @@ inline double wave_cost(int M, int N, int K, int sms, int bn) {
 
 inline int pick_block_n_split(int M, int N, int K, int sms) {
   return wave_cost(M, N, K, sms, 256) <= wave_cost(M, N, K, sms, 128) ? 256 : 128;
+}
+
+// Host: the output map of a staged epilogue.
+inline int make_staged_map(CUtensorMap* tmC, const void* C, int M, int N, long long ldc) {
+  return encode_tmap_2d(tmC, C, 2, (uint64_t)N, (uint64_t)M, (uint64_t)ldc * 2, 64, 32, 1);
 }
 
 // Host: tensor maps for the two operands.

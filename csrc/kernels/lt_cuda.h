@@ -107,6 +107,8 @@ int lt_gemm_typed(int kind, const void* A, const void* B, void* C, int M, int N,
 int lt_gemm_e4m3(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
                  long long ldc, int out_fp32, const float* a_scale, const float* b_scale, const void* bias,
                  const void* residual, long long ldr, int act, float alpha, void* stream);
+int lt_gemm_staged(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb, long long ldc, int act,
+                   float alpha, int block_n, void* stream);
 int lt_gemm_block_diag(const void* A, const void* B, float* C, int M, int blocks, int nb, int K, long long lda,
                        long long ldc, void* stream);
 
@@ -197,7 +199,7 @@ int lt_latent_decode(const void* q, const void* cache, const int* tables, const 
 int lt_moe_plan(const float* logits, const float* correction, float* weight, int* slot, int* src, int* group, int* group_rows, int* live,
                 void* pairs, int* counts, const void* x, void* xs, int row_bytes, int N, int E, int top, int block_rows, void* stream);
 int lt_moe_grouped_gemm(const void* A, const void* W, void* C, const int* group, const int* live, int max_blocks, int experts, int N,
-                        int K, void* stream);
+                        int K, int act, void* stream);
 
 // ---- gemm_simt.cu: CUDA-core GEMM (true fp32, odd shapes, batches) and narrow projections with fp32 results
 int lt_gemm_simt(int in_fp32, int out_fp32, const void* A, const void* B, void* C, int M, int N, int K, long long lda,

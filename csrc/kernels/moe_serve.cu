@@ -183,29 +183,30 @@ __global__ void __launch_bounds__(256) moe_place_kernel(const int2* __restrict__
   if (blockIdx.x == 0) write_groups(p, cnt, first, total, E, block_rows);
 }
 
-// C[slots, N] = A[slots, K] @ W[expert of the slot's 128-row block]^T; only the blocks in use are computed.
-template <int BLOCK_N>
+// C[slots, N] = A[slots, K] @ W[expert of the slot's 128-row block]^T, gated or not; only the blocks in use are computed.
+template <int BLOCK_N, int EPI>
 __global__ void __launch_bounds__(kGemmThreads, 1)
-moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const GemmParams p,
-                        const int* __restrict__ live) {
+moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
+                        const __grid_constant__ CUtensorMap tmC, const GemmParams p, const int* __restrict__ live) {
   __shared__ GemmParams q;
   if (threadIdx.x == 0) {
     q = p;
     q.dp_tiles = min(p.num_tiles, *live * p.n_blocks);
   }
   __syncthreads();
-  gemm_body<BLOCK_N, 0, 0>(&tmA, &tmB, q, NoGate(), NoDone());
+  gemm_body<BLOCK_N, 0, 0, 0, false, EPI>(&tmA, &tmB, q, NoGate(), NoDone(), 0, &tmC);
 }
 
-template <int BLOCK_N>
-static int launch_grouped(const CUtensorMap& tmA, const CUtensorMap& tmB, const GemmParams& p, const int* live, int grid, cudaStream_t st) {
+template <int BLOCK_N, int EPI>
+static int launch_grouped(const CUtensorMap& tmA, const CUtensorMap& tmB, const CUtensorMap& tmC, const GemmParams& p, const int* live,
+                          int grid, cudaStream_t st) {
   static bool configured = false;
-  auto kern = moe_grouped_gemm_kernel<BLOCK_N>;
+  auto kern = moe_grouped_gemm_kernel<BLOCK_N, EPI>;
   if (!configured) {
-    LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, GemmCfg<BLOCK_N>::kSmemBytes));
+    LT_RETURN_IF_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, GemmCfg<BLOCK_N>::kStagedSmemBytes));
     configured = true;
   }
-  kern<<<grid, kGemmThreads, GemmCfg<BLOCK_N>::kSmemBytes, st>>>(tmA, tmB, p, live);
+  kern<<<grid, kGemmThreads, GemmCfg<BLOCK_N>::kStagedSmemBytes, st>>>(tmA, tmB, tmC, p, live);
   LT_LAUNCH_CHECK();
   return 0;
 }
@@ -257,29 +258,34 @@ int lt_moe_plan(const float* logits, const float* correction, float* weight, int
   return 0;
 }
 
-// C [max_blocks * 128, N] bf16 = A @ W[group[block]]^T for the first *live blocks of 128 rows; W [experts, N, K]; K and N multiples of 8.
+// C [max_blocks * 128, N] bf16 = A @ W[group[block]]^T for the first *live blocks of 128 rows; K and N multiples of 8.  act 0: W [experts,
+// N, K]; 1 (GELU) or 2 (SiLU): W [experts, 2 N, K], gate rows, then up rows, and C = act(gate) * up.
 int lt_moe_grouped_gemm(const void* A, const void* W, void* C, const int* group, const int* live, int max_blocks, int experts, int N,
-                        int K, void* stream) {
+                        int K, int act, void* stream) {
   using namespace lt;
-  if (max_blocks < 1 || (K & 7) || (N & 7)) return -int(kStatusBadArgument);
-  const int slots = max_blocks * kBlockM, sms = sm_count();
-  const int block_n = pick_block_n(slots, N, sms);
+  if (max_blocks < 1 || (K & 7) || (N & 7) || act < 0 || act > 2) return -int(kStatusBadArgument);
+  const int slots = max_blocks * kBlockM, sms = sm_count(), rows = act ? 2 * N : N;
+  const int block_n = act ? 256 : pick_block_n(slots, N, sms);
+  const int out_n = act ? 128 : block_n;
   GemmParams p{};
   p.M = slots; p.N = N; p.K = K;
   p.C = C; p.ldc = N; p.alpha = 1.f;
+  p.glu_act = act;
   p.status = device_status_word();
-  fill_tiles(p, block_n);
+  fill_tiles(p, out_n);
   p.raster = 2;
   p.group_of_mblk = group;
-  p.b_group_rows = N;
-  CUtensorMap tmA, tmB;
-  int r = encode_tmap_2d(&tmA, A, 2, (uint64_t)K, (uint64_t)slots, (uint64_t)K * 2, kBlockK, kBlockM, 1);
-  if (r) return 1000 + r;
-  r = encode_tmap_2d(&tmB, W, 2, (uint64_t)K, (uint64_t)experts * N, (uint64_t)K * 2, kBlockK, block_n, 1);
-  if (r) return 2000 + r;
+  p.b_group_rows = rows;
+  CUtensorMap tmA, tmB, tmC;
+  int r = make_operand_maps(&tmA, &tmB, A, W, slots, experts * rows, K, K, K, 0, 0, out_n);
+  if (r) return r;
+  r = make_staged_map(&tmC, C, slots, N, N);
+  if (r) return 3000 + r;
   const int grid = sms < p.num_tiles ? sms : p.num_tiles;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return block_n == 256 ? launch_grouped<256>(tmA, tmB, p, live, grid, st) : launch_grouped<128>(tmA, tmB, p, live, grid, st);
+  if (act) return launch_grouped<256, kEpiGlu>(tmA, tmB, tmC, p, live, grid, st);
+  return block_n == 256 ? launch_grouped<256, kEpiStaged>(tmA, tmB, tmC, p, live, grid, st)
+                        : launch_grouped<128, kEpiStaged>(tmA, tmB, tmC, p, live, grid, st);
 }
 
 }  // extern "C"

@@ -21,7 +21,8 @@ _SIGS = {
     "lt_latent_decode": [_vp] * 7 + [_i] * 9 + [_f, _vp],
     "lt_flash_fwd_shared": [_vp] * 6 + [_i] * 5 + [_ll] * 4 + [_f, _i, _vp],
     "lt_moe_plan": [_vp] * 12 + [_i] * 5 + [_vp],
-    "lt_moe_grouped_gemm": [_vp] * 5 + [_i] * 4 + [_vp],
+    "lt_moe_grouped_gemm": [_vp] * 5 + [_i] * 5 + [_vp],
+    "lt_gemm_staged": [_vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _i, _f, _i, _vp],
     "lt_gemm_skinny_glu": [_vp, _ll, _vp, _vp, _i, _i, _i, _i, _vp],
     "lt_gemm_skinny_batch": [_vp, _ll, _ll, _vp, _vp, _ll, _ll, _i, _i, _i, _i, _vp],
     "lt_gemm_skinny_grouped": [_vp, _ll] + [_vp] * 6 + [_i] * 5 + [_vp],
@@ -823,6 +824,9 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None, alpha: float = 1.0)
     if M == 0:
         return torch.empty((0, N), dtype=out_dtype, device=x.device)
     if x.dtype == torch.bfloat16 and Kd % 8 == 0 and (M == 1 or x.stride(0) % 8 == 0) and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
+        if M > 128 and Kd <= 2048 and N >= 512 and N % 8 == 0 and out_dtype == torch.bfloat16:
+            # a short K loop is bound by how its results leave; a narrow tile where wide ones would not fill the GPU
+            return gemm_staged(x, w, alpha=alpha, block_n=256 if (M + 127) // 128 * ((N + 255) // 256) >= 100 else 128)
         return gemm(x, w, out_dtype=out_dtype, alpha=alpha)
     y = torch.empty((M, N), dtype=out_dtype, device=x.device)
     rc = _fn("lt_gemm_simt")(_f32(x), _f32(y), x.data_ptr(), w.data_ptr(), y.data_ptr(), M, N, Kd, x.stride(0), Kd, N, 1, 0, 0, 0,
@@ -1123,8 +1127,20 @@ def act_glu(gu, act: str, live=None, block_rows: int = 0):
     return h
 
 
+def gemm_staged(a, b, *, act: str = "", alpha: float = 1.0, block_n: int = 0):
+    """alpha * a [M, K] @ b [N, K]^T in bf16, the result leaving through shared memory and TMA; with act, b holds gate rows, then up rows,
+    and the result is act(gate) * up."""
+    (M, Kd), N = a.shape, b.shape[0] // 2 if act else b.shape[0]
+    assert a.dtype == b.dtype == torch.bfloat16 and a.stride(1) == 1 and b.stride(1) == 1 and b.shape[1] == Kd
+    y = torch.empty((M, N), dtype=a.dtype, device=a.device)
+    rc = _fn("lt_gemm_staged")(a.data_ptr(), b.data_ptr(), y.data_ptr(), M, N, Kd, a.stride(0), b.stride(0), N, _ACT[act] if act else 0, float(alpha),
+                               block_n, _stream())
+    _check(rc, "lt_gemm_staged")
+    return y
+
+
 def glu_mlp(x, gu, down, act: str):
-    """down @ (act(gate @ x) * (up @ x)) with gu = [gate; up]; up to 128 rows of bf16 gate in the product's epilogue."""
+    """down @ (act(gate @ x) * (up @ x)) with gu = [gate; up]; bf16 gates in the first product's epilogue."""
     M, Kd = x.shape
     F = gu.shape[0] // 2
     if x.dtype == torch.bfloat16 and 0 < M <= 128 and Kd % 32 == 0 and F % 8 == 0 and x.stride(0) % 8 == 0 and _aligned(x, gu):
@@ -1132,6 +1148,8 @@ def glu_mlp(x, gu, down, act: str):
         rc = _fn("lt_gemm_skinny_glu")(x.data_ptr(), x.stride(0), gu.data_ptr(), h.data_ptr(), M, F, Kd, _ACT[act], _stream())
         _check(rc, "lt_gemm_skinny_glu")
         return linear(h, down)
+    if x.dtype == torch.bfloat16 and M > 128 and Kd % 8 == 0 and F % 8 == 0 and x.stride(0) % 8 == 0 and _aligned(x, gu):
+        return linear(gemm_staged(x, gu, act=act), down)
     return linear(act_glu(linear(x, gu), act), down)
 
 
@@ -1169,11 +1187,12 @@ def moe_grouped(x, w, plan, act: str = "", picked: bool = False):
     src = plan["src"] if picked else None
     if br == 128:
         assert x.is_contiguous() and not picked
-        y = torch.empty((M, N), dtype=x.dtype, device=dev)
-        rc = _fn("lt_moe_grouped_gemm")(x.data_ptr(), w.data_ptr(), y.data_ptr(), plan["group"].data_ptr(), plan["live"].data_ptr(), plan["blocks"], E, N,
-                                        Kd, _stream())
+        n = N // 2 if act else N
+        y = torch.empty((M, n), dtype=x.dtype, device=dev)
+        rc = _fn("lt_moe_grouped_gemm")(x.data_ptr(), w.data_ptr(), y.data_ptr(), plan["group"].data_ptr(), plan["live"].data_ptr(), plan["blocks"], E, n,
+                                        Kd, _ACT[act] if act else 0, _stream())
         _check(rc, "lt_moe_grouped_gemm")
-        return act_glu(y, act, plan["live"], br) if act else y
+        return y
     if x.dtype == torch.bfloat16 and plan["mma"]:
         n = N // 2 if act else N
         y = torch.empty((M, n), dtype=x.dtype, device=dev)

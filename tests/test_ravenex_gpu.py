@@ -289,6 +289,18 @@ def test_gated_feed_forward(dtype, act, M, W, F):
     _close(K.act_glu(big, act), f(_d(big)[:, :F]) * _d(big)[:, F:], dtype)
 
 
+@pytest.mark.parametrize("M,N,Kd", [(129, 8, 64), (300, 72, 40), (128, 256, 512), (1000, 1000, 264), (257, 2056, 2048), (40, 64, 8)])
+def test_products_with_a_staged_epilogue(M, N, Kd):
+    K = _k()
+    x, w = _rand(M, Kd + 8, dtype=BF, seed=1)[:, :Kd], _rand(2 * N, Kd, dtype=BF, seed=2, scale=2 * Kd ** -0.5)
+    want = _d(x) @ _d(w).t()
+    for bn in (0, 128, 256):
+        _close(K.gemm_staged(x, w[:N], alpha=0.5, block_n=bn), 0.5 * want[:, :N], BF)
+    for act, f in (("gelu", R.gelu), ("silu", R.silu)):
+        _close(K.gemm_staged(x, w, act=act), f(want[:, :N]) * want[:, N:], BF)
+    assert K.status_fetch() == 0
+
+
 @pytest.mark.parametrize("dtype", DT)
 def test_token_gate(dtype):
     K = _k()
