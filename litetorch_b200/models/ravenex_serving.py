@@ -25,6 +25,7 @@ class RavenexModel(ServingModel):
         # the pages of a layer hold a latent and the rotated key part as one key of one head; there are no values beside it
         self.cache = PagedKVCache.per_layer([None if lay.mix.c_norm is None else (1, lay.mix.c + lay.mix.r, 0) for lay in engine.layers],
                                             num_blocks, block_size, engine.device, engine.dtype)
+        self.page_copies = block_size in (8, 16) or block_size % 32 == 0          # what the decode kernel on latents copies whole
         self.source = [i if lay.cfg.mixer.kv_from is None else lay.cfg.mixer.kv_from for i, lay in enumerate(engine.layers)]
         # per layer with latents: the windows of the layers that want them unrolled in prompts
         self.windows = {j: [lay.cfg.mixer.window for i, lay in enumerate(engine.layers) if self.source[i] == j and lay.mix.tensor_cores]
@@ -135,7 +136,7 @@ class RavenexModel(ServingModel):
             a, w = lay.cfg.mixer, lay.mix
 
             def attend(q, kc):
-                if w.tensor_cores:
+                if w.tensor_cores and self.page_copies:
                     keys = min(a.window, width * self.block_size) if a.window > 0 else width * self.block_size
                     return K.latent_decode(q, kc, tables, ctx, rank=w.c, window=a.window, scale=a.scale, max_keys=keys)
                 return K.window_attn(q, kc, kc, tables, pos, D=w.c + w.r, E=w.c, window=a.window, scale=a.scale)

@@ -63,13 +63,13 @@ class Suite:
         with torch.no_grad():
             return self.forward(cfg, w, toks)
 
-    def check_portions(self, name, device, dtype, length, schedules):
+    def check_portions(self, name, device, dtype, length, schedules, block_size=16):
         """Whole prompts, portions and single tokens all give the logits of the plain statement."""
         cfg = self.configs[name]
         w = self.weights(cfg)
         toks = tokens(cfg, length, 1)
         want = self.reference(cfg, w, toks)
-        model, sched = server(self.engine(cfg, w, device, dtype), blocks=2 * (length // 16 + 2))
+        model, sched = server(self.engine(cfg, w, device, dtype), blocks=2 * (length // block_size + 2), block_size=block_size)
         for n, cuts in enumerate(schedules):
             e = self.measure(run_portions(model, sched, n, toks, cuts), want, cfg, dtype)
             assert e < TOL[dtype], (name, cuts, e)

@@ -319,6 +319,12 @@ def test_portions_of_all_sizes_match_the_plain_statement(name, dtype):
     assert _k().status_fetch() == 0
 
 
+@pytest.mark.parametrize("block_size", [1, 8, 24, 32, 96])
+@pytest.mark.parametrize("name", ["mixed", "tiles"])
+def test_block_sizes(name, block_size):
+    U.SUITE.check_portions(name, "cuda", BF, 210, [[210], [100, 1]], block_size)
+
+
 @pytest.mark.parametrize("dtype", DT)
 @pytest.mark.parametrize("name", ["mixed", "tiles", "choice"])
 def test_requests_side_by_side_and_reused_pages(name, dtype):
@@ -367,11 +373,11 @@ def test_results_do_not_depend_on_pages():
     eng = U.engine(cfg, w, "cuda", BF)
     toks = U.tokens(cfg, 150, 5)
     outs = []
-    for bs, others in ((16, 0), (16, 2), (32, 1)):
+    for bs, others in ((16, 0), (16, 2), (32, 1), (96, 1)):
         model, sched = U.server(eng, blocks=64, slots=4, block_size=bs)
         for o in range(others):
             sched.feed(model, [(50 + o, U.tokens(cfg, 40 + o, o), [])])
         if others == 2:
             sched.end_session(50)
         outs.append(U.run_portions(model, sched, 0, toks, [60, 1, 1, 50, 1]))
-    assert torch.equal(outs[0], outs[1]) and torch.equal(outs[0], outs[2])
+    assert all(torch.equal(outs[0], o) for o in outs[1:])
