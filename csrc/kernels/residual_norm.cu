@@ -66,18 +66,43 @@ __global__ void __launch_bounds__(max_threads(V)) residual_norm_kernel(const Res
       if (yr) load(yr + c, y[i]);
     }
   }
+  // Few rows leave every load's latency in the open: there the norms' weights, and eight expert rows at a time, are on their way
+  // together.  (With many rows that costs more in registers than it hides.)
+  constexpr bool kEarly = NC == 1;
+  [[maybe_unused]] float wy[V], wn[V];
+  if constexpr (kEarly) {
+    const int c = threadIdx.x * V;
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      wy[v] = p.y_norm && c + v < W ? p.y_norm[c + v] : 1.f;
+      wn[v] = p.norm && c + v < W ? p.norm[c + v] : 1.f;
+    }
+  }
   if (p.z) {
-    for (int j = 0; j < p.top; ++j) {
-      const T* zr = static_cast<const T*>(p.z) + (long long)p.z_slot[row * p.top + j] * W;
-      const float a = p.z_weight[row * p.top + j];
+    constexpr int kRows = kEarly ? 8 : 1;
+    for (int j0 = 0; j0 < p.top; j0 += kRows) {
+      const T* zr[kRows];
+      float a[kRows];
+#pragma unroll
+      for (int j = 0; j < kRows; ++j) {
+        const bool in = j0 + j < p.top;
+        zr[j] = static_cast<const T*>(p.z) + (in ? (long long)p.z_slot[row * p.top + j0 + j] * W : 0);
+        a[j] = in ? p.z_weight[row * p.top + j0 + j] : 0.f;
+      }
 #pragma unroll
       for (int i = 0; i < NC; ++i) {
         const int c = (i * nt + threadIdx.x) * V;
         if (c < W) {
-          float z[V];
-          load(zr + c, z);
+          float z[kRows][V];
 #pragma unroll
-          for (int v = 0; v < V; ++v) y[i][v] = fmaf(a, z[v], y[i][v]);
+          for (int j = 0; j < kRows; ++j)
+            if (j0 + j < p.top) load(zr[j] + c, z[j]);
+#pragma unroll
+          for (int j = 0; j < kRows; ++j)
+            if (j0 + j < p.top) {
+#pragma unroll
+              for (int v = 0; v < V; ++v) y[i][v] = fmaf(a[j], z[j][v], y[i][v]);
+            }
         }
       }
     }
@@ -97,7 +122,10 @@ __global__ void __launch_bounds__(max_threads(V)) residual_norm_kernel(const Res
       const int c = (i * nt + threadIdx.x) * V;
       if (c < W) {
 #pragma unroll
-        for (int v = 0; v < V; ++v) x[i][v] = fmaf(f, p.y_norm ? y[i][v] * p.y_norm[c + v] : y[i][v], x[i][v]);
+        for (int v = 0; v < V; ++v) {
+          if constexpr (kEarly) x[i][v] = fmaf(f, y[i][v] * wy[v], x[i][v]);
+          else x[i][v] = fmaf(f, p.y_norm ? y[i][v] * p.y_norm[c + v] : y[i][v], x[i][v]);
+        }
       }
     }
   }
@@ -128,7 +156,10 @@ __global__ void __launch_bounds__(max_threads(V)) residual_norm_kernel(const Res
     if (c < W) {
       float o[V];
 #pragma unroll
-      for (int v = 0; v < V; ++v) o[v] = p.norm ? x[i][v] * inv * p.norm[c + v] : x[i][v];
+      for (int v = 0; v < V; ++v) {
+        if constexpr (kEarly) o[v] = x[i][v] * inv * wn[v];
+        else o[v] = p.norm ? x[i][v] * inv * p.norm[c + v] : x[i][v];
+      }
       if constexpr (V == 4) stf4(h + c, make_float4(o[0], o[1], o[2], o[3]));
       else stf(h + c, o[0]);
     }

@@ -1,4 +1,4 @@
-"""Text generation from a model directory (config.json + *.safetensors: a Hugging Face Llama, a Safuvik, any family of
+"""Text generation from a model directory (config.json + *.safetensors: a Hugging Face Llama, a Safuvik, a Ravenex, any family of
 `models.registry`) on the serving path of this package: continuous batching over a paged KV cache, CUDA-graph decode steps.
 
     python examples/generate_llama.py --model /models/llama --sentencepiece /models/llama/tokenizer.model \
