@@ -143,25 +143,24 @@ __device__ __forceinline__ void ld_mma(float (&d)[4], const uint32_t (&a)[4], ui
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// Barriers of the eight warps that make the scores.
+// Barrier of the eight warps that make the scores: true where all of them say so.
 __device__ __forceinline__ bool ld_bar_and(bool v) {
   int r;
   asm volatile("{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbar.red.and.pred q, 1, 256, p;\nselp.s32 %0, 1, 0, q;\n}" : "=r"(r) : "r"(int(v)) : "memory");
   return r != 0;
 }
 
-// Shared memory of a CTA: slack for alignment, tiles (later the outputs of the split), score quarters, weights, per-head numbers,
-// barriers.
+// Shared memory of a CTA: slack for alignment, tiles, score quarters, weights, per-head numbers, barriers.
 __host__ __device__ inline int ld_smem_bytes(int w, int heads, int stages) {
   return 1024 + stages * kLdKeys * w * 2 + 2 * (4 * heads * kLdSPitch * 4 + heads * kLdPPitch * 2 + heads * 4) + 2 * heads * 4 +
          (2 * kLdMaxStages + 4) * 8;
 }
 
-// MT: 16-head blocks of a CTA (1 or 2).  FULL: the largest row (w 576, c 512),
-// whose loops have no conditions, so that loads run ahead of the products.
+// MT: 16-head blocks of a CTA (1 or 2).  FULL: the largest row (w 576, c 512), whose loops have no conditions, so that loads run
+// ahead of the products.
 template <int MT, bool FULL>
-__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap tmap,
-                                                                               const LatentDecodeParams p) {
+__global__ void __launch_bounds__(kLdThreads, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmap, const LatentDecodeParams p) {
   constexpr int MH = MT * 16;
   constexpr int TPH = kLdRole / MH;              // threads per head in the softmax
   constexpr int KPT = kLdKeys / TPH;             // keys of each
